@@ -58,6 +58,7 @@ struct DecParams {
   const float* sinks;   // per head, or null: exp(sink) joins the denominator (no key, no value)
   const float* gate;    // float logits [S, gate_ld] or null: head h's output times sigmoid(gate[seq, h])
   int gate_ld;
+  SoftCap cap;          // cap.c > 0: scores are bounded, cap tanh(score / cap), before mask and softmax (the sink is not)
 };
 
 // The last step of a row: the sink joins the denominator, the sum is divided, the gate applied.
@@ -236,6 +237,7 @@ attn_decode_kernel(const DecParams p) {
     for (int i = 0; i < DTILES; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
     float mA = -INFINITY, mB = -INFINITY, lA = 0.f, lB = 0.f;
     const int mat = lane >> 3, rr = lane & 7;
+    const float sl = p.cap.c > 0.f ? 1.f : p.scale_log2e;
 
     for (int i = warp; i < n_tiles; i += NW) {
       cp_async_wait<D - 1>();                       // this warp's oldest group, tile i, has landed
@@ -261,6 +263,13 @@ attn_decode_kernel(const DecParams p) {
         for (int np = 0; np < TILE / 16; ++np) {
           mma16816(sc[2 * np], qf[kk], kf[kk][np][0], kf[kk][np][1]);
           mma16816(sc[2 * np + 1], qf[kk], kf[kk][np][2], kf[kk][np][3]);
+        }
+      }
+      if (p.cap.c > 0.f) {                             // bounded scores leave the bound in the log2 domain (sl is 1 then)
+#pragma unroll
+        for (int nt = 0; nt < TILE / 8; ++nt) {
+          sc[nt][0] = softcap_log2(sc[nt][0], p.cap); sc[nt][1] = softcap_log2(sc[nt][1], p.cap);
+          if (G > 8) { sc[nt][2] = softcap_log2(sc[nt][2], p.cap); sc[nt][3] = softcap_log2(sc[nt][3], p.cap); }
         }
       }
       // ---- the V fragments are asked for now and used after the softmax arithmetic
@@ -293,7 +302,7 @@ attn_decode_kernel(const DecParams p) {
       mxB = fmaxf(mxB, __shfl_xor_sync(0xffffffffu, mxB, 1));
       mxB = fmaxf(mxB, __shfl_xor_sync(0xffffffffu, mxB, 2));
       // running maximum in the exp2 domain (the scale is positive, so it commutes with max)
-      const float mnA = fmaxf(mA, mxA * p.scale_log2e), mnB = fmaxf(mB, mxB * p.scale_log2e);
+      const float mnA = fmaxf(mA, mxA * sl), mnB = fmaxf(mB, mxB * sl);
       const float useA = (mnA == -INFINITY) ? 0.f : mnA, useB = (mnB == -INFINITY) ? 0.f : mnB;
       if (__any_sync(0xffffffffu, mnA != mA || mnB != mB)) {      // a new maximum somewhere: rescale
         const float corrA = fast_exp2(mA - useA), corrB = fast_exp2(mB - useB);     // exp2(-inf) = 0
@@ -306,7 +315,6 @@ attn_decode_kernel(const DecParams p) {
       for (int kb = 0; kb < TILE / 16; ++kb) {
         uint32_t a[4];
         {
-          const float sl = p.scale_log2e;
           const float p0 = fast_exp2(fmaf(sc[2 * kb][0], sl, -useA)), p1 = fast_exp2(fmaf(sc[2 * kb][1], sl, -useA));
           const float p2 = fast_exp2(fmaf(sc[2 * kb][2], sl, -useB)), p3 = fast_exp2(fmaf(sc[2 * kb][3], sl, -useB));
           const float p4 = fast_exp2(fmaf(sc[2 * kb + 1][0], sl, -useA)), p5 = fast_exp2(fmaf(sc[2 * kb + 1][1], sl, -useA));
@@ -438,13 +446,13 @@ int launch_dec(const DecParams& p, int num_seqs, cudaStream_t s) {
 // kcache / vcache: [num_pages][nkv][page_size][hd] bf16. kv_lens [S]: keys visible to each
 // sequence's token (its own included). splits: ranges of keys per sequence (1..16, one cluster).
 // chunk > 0: only the keys of the token's own block of `chunk` positions; sinks float [nh] or null; gate float
-// logits [S, gate_ld] or null (see DecParams).
+// logits [S, gate_ld] or null; softcap > 0: bounded scores (see DecParams).
 // `err` is not used (this kernel has no wait that can run out); it keeps the launchers alike.
 RLLM_API int rllm_attention_decode(const void* q, int q_stride, const void* kcache, const void* vcache,
                                    long long num_pages, void* out, int out_stride, const int* kv_lens,
                                    const int* block_table, int bt_stride, int num_seqs, int nh, int nkv, int hd,
                                    int page_size, float scale, int window, int chunk, const float* sinks,
-                                   const float* gate, int gate_ld, int splits, int* err, void* stream) {
+                                   const float* gate, int gate_ld, float softcap, int splits, int* err, void* stream) {
   (void)err;
   if (num_seqs <= 0) return 0;
   if ((hd != 64 && hd != 128) || nkv <= 0 || nh % nkv || nh / nkv > 16) return ERR_BAD_SIZE;
@@ -457,6 +465,7 @@ RLLM_API int rllm_attention_decode(const void* q, int q_stride, const void* kcac
   p.kv_lens = kv_lens; p.block_table = block_table; p.bt_stride = bt_stride; p.nh = nh; p.nkv = nkv;
   p.page_size = page_size; p.window = window; p.splits = splits; p.scale_log2e = scale * 1.4426950408889634f;
   p.chunk = chunk; p.sinks = sinks; p.gate = gate; p.gate_ld = gate_ld;
+  p.cap = make_softcap(softcap, scale);
   p.page_shift = -1;
   for (int sft = 0; sft < 31; ++sft) if ((1 << sft) == page_size) p.page_shift = sft;
   cudaStream_t s = (cudaStream_t)stream;

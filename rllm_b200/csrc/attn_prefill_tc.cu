@@ -97,6 +97,8 @@ struct PfParams {
   int sigmoid;           // != 0: weights sigmoid(score + bias), not normalised
   const float* gate;     // float logits [T, gate_ld] or null: head h's output times sigmoid(gate[t, h])
   int gate_ld;
+  SoftCap cap;           // cap.c > 0: scores are bounded, cap tanh(score / cap), before mask and softmax (the sink is not)
+  float cap_z;           // scale / cap
   int box_rows;          // TMA variant: keys per copy = min(page size, 128)
   int row_pairs, num_seqs, sm_count;
   float scale_log2e;
@@ -128,6 +130,37 @@ template <int N> __device__ __forceinline__ void cp_async_wait() {
 // instruction descriptor: bf16 x bf16 -> f32, A K-major, B K-major or MN-major
 __host__ __device__ constexpr uint32_t idesc(int M, int N, bool b_mn_major) {
   return umma_idesc_bf16(M, N) | (b_mn_major ? (1u << 16) : 0u);
+}
+
+// Two scores at a time: x = (x0, x1), bounded, in the log2 domain. tanh(z) = z P(z^2) on |z| <= 1 with a polynomial of
+// degree 6 (interpolated at the Chebyshev points of [0, 1] in z^2: 4e-8 from tanh before rounding), which runs on the FMA
+// pipe and leaves the transcendental unit to the softmax.
+__device__ __forceinline__ uint64_t f32x2(float a, float b) {
+  uint64_t d;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(a), "f"(b));
+  return d;
+}
+__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
+  uint64_t d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+  return d;
+}
+__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
+  uint64_t d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
+__device__ __forceinline__ void softcap_poly2(uint32_t& x0, uint32_t& x1, float zscale, float c) {
+  const uint64_t z = mul2(f32x2(__uint_as_float(x0), __uint_as_float(x1)), f32x2(zscale, zscale));
+  const uint64_t t = mul2(z, z);
+  uint64_t q = fma2(t, f32x2(0.0010380251f, 0.0010380251f), f32x2(-0.00619432483f, -0.00619432483f));
+  q = fma2(q, t, f32x2(0.0202797083f, 0.0202797083f));
+  q = fma2(q, t, f32x2(-0.0534516464f, -0.0534516464f));
+  q = fma2(q, t, f32x2(0.133250761f, 0.133250761f));
+  q = fma2(q, t, f32x2(-0.33332828f, -0.33332828f));
+  q = fma2(q, t, f32x2(0.999999949f, 0.999999949f));
+  const uint64_t r = mul2(mul2(z, f32x2(c, c)), q);
+  asm("mov.b64 {%0, %1}, %2;" : "=r"(x0), "=r"(x1) : "l"(r));
 }
 
 // TMA: the K and V tiles come by tensor copies over the caches seen as [pages * kv heads][page size][HD].
@@ -433,7 +466,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_
     const uint32_t pv_addr = lane_addr + C::O_COL + (uint32_t)g * HD;
     const uint32_t prow = p_s + (uint32_t)g * C::P_BYTES + (uint32_t)(r * 128);
     constexpr int NC = PN / 32;                           // the row's scores come 32 at a time
-    const float sl = p.scale_log2e;
+    const bool bounded = p.cap.c > 0.f;
+    const float sl = bounded ? 1.f : p.scale_log2e;        // bounded scores leave the bound in the log2 domain
     // m: what the exponentials are taken against, up to 2^8 behind the true maximum. A sink opens the row's
     // running softmax as a key of score `sink` (not scaled) and value zero.
     const bool sig = p.sigmoid != 0;
@@ -463,6 +497,29 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_
       tc_fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive(&s_free[k % SB]);        // the accumulator may take the scores of step k + 3
+      if (bounded) {
+        float far[NC];
+#pragma unroll
+        for (int c = 0; c < NC; ++c) {
+          far[c] = 0.f;
+#pragma unroll
+          for (int i = 0; i < 32; i += 2) far[c] = fmax3(far[c], fabsf(__uint_as_float(v[c][i])), fabsf(__uint_as_float(v[c][i + 1])));
+        }
+        float mz = far[0];
+#pragma unroll
+        for (int c = 1; c < NC; ++c) mz = fmaxf(mz, far[c]);
+        if (__all_sync(0xffffffffu, mz * fabsf(p.cap_z) <= 1.f)) {        // every score of the warp's rows within the bound
+#pragma unroll
+          for (int c = 0; c < NC; ++c)
+#pragma unroll
+            for (int i = 0; i < 32; i += 2) softcap_poly2(v[c][i], v[c][i + 1], p.cap_z, p.cap.c);
+        } else {
+#pragma unroll
+          for (int c = 0; c < NC; ++c)
+#pragma unroll
+            for (int i = 0; i < 32; ++i) v[c][i] = __float_as_uint(softcap_log2(__uint_as_float(v[c][i]), p.cap));
+        }
+      }
       if (!valid || j0 + PN - 1 > pos || (j0 < lo && j0 + PN > kf)) {        // some key is hidden from this row
 #pragma unroll
         for (int c = 0; c < NC; ++c)
@@ -642,13 +699,13 @@ int launch_pf(const CUtensorMap& mk, const CUtensorMap& mv, const PfParams& p, i
 // max_q_len: the longest portion in the batch (sizes the list of work items). Head sizes 64 and 128.
 // chunk > 0: a query sees only the keys of its own block of `chunk` positions (blocks counted from position 0);
 // sinks: float [nh] or null; gate: float logits [T, gate_ld] or null (see PfParams); keep_first, sigmoid: see PfParams.
-// sm_count: CTAs to launch at most (0: asked from the device).
+// softcap > 0: bounded scores. sm_count: CTAs to launch at most (0: asked from the device).
 RLLM_API int rllm_attention_prefill_tc(const void* q, int q_stride, const void* kcache, const void* vcache,
                                        void* out, int out_stride, const int* cu_q, const int* kv_lens,
                                        const int* block_table, int bt_stride, int num_seqs, int max_q_len,
                                        int num_pages, int nh, int nkv, int hd, int page_size, float scale, int window,
                                        int chunk, const float* sinks, const float* gate, int gate_ld,
-                                       int keep_first, int sigmoid, int* err, int sm_count, void* stream) {
+                                       int keep_first, int sigmoid, float softcap, int* err, int sm_count, void* stream) {
   if (num_seqs <= 0 || max_q_len <= 0) return 0;
   if ((hd != 64 && hd != 128) || nkv <= 0 || nh % nkv || page_size <= 0 || num_pages <= 0 || keep_first < 0 || scale <= 0.f)
     return ERR_BAD_SIZE;
@@ -661,6 +718,7 @@ RLLM_API int rllm_attention_prefill_tc(const void* q, int q_stride, const void* 
   p.page_shift = -1;
   if ((page_size & (page_size - 1)) == 0) { p.page_shift = 0; while ((1 << p.page_shift) < page_size) ++p.page_shift; }
   p.chunk = chunk; p.sinks = sinks; p.gate = gate; p.gate_ld = gate_ld; p.keep_first = keep_first; p.sigmoid = sigmoid;
+  p.cap = make_softcap(softcap, scale); p.cap_z = softcap > 0.f ? scale / softcap : 0.f;
   p.window = window; p.scale_log2e = scale * 1.4426950408889634f; p.err = err;
   const int G = nh / nkv;
   p.row_pairs = (max_q_len * G + RT * PM - 1) / (RT * PM); p.num_seqs = num_seqs;

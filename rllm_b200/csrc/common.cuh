@@ -63,6 +63,24 @@ __device__ __forceinline__ float block_max(float v, float* red) {
   return r;
 }
 
+// A bounded score in the log2 domain, cap log2(e) tanh(raw scale / cap) = c - 2 c / (1 + 2^(raw k)) with c = cap log2(e)
+// and k = 2 log2(e) scale / cap: one exponential and one reciprocal, exact to a few units in the last place of c
+// (2^(+-inf) gives +-c).
+struct SoftCap {
+  float k, c;                     // c = 0: no bound
+};
+static inline SoftCap make_softcap(float softcap, float scale) {
+  SoftCap s = {0.f, 0.f};
+  if (softcap > 0.f) { s.k = 2.f * 1.4426950408889634f * scale / softcap; s.c = softcap * 1.4426950408889634f; }
+  return s;
+}
+__device__ __forceinline__ float softcap_log2(float raw, const SoftCap& s) {
+  float e, r;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(raw * s.k));
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.f + e));
+  return fmaf(-2.f * s.c, r, s.c);
+}
+
 static inline int launch_status() {
   cudaError_t e = cudaPeekAtLastError();
   if (e != cudaSuccess) { cudaGetLastError(); return (int)e; }

@@ -237,9 +237,9 @@ RLLM_API int rllm_rmsnorm(const float* x, const int* rows, const void* w, int w_
 // Cache layout: [page][kv head][offset in page][hd].
 // Reference: src/gpu/cuda/shaders/rope.cu:62-77 and attention.cu:295-300.
 // The rotation of a step, made once and read by every layer: cs[t][i] = (cos, sin)(positions[t] *
-// inv_freq[i]) in float, i < n_freq. The same sincosf the kernels below call when they get no table.
+// inv_freq[i]) * mag in float, i < n_freq. The same sincosf the kernels below call when they get no table.
 __global__ void rope_table_kernel(const int* __restrict__ positions, const float* __restrict__ inv_freq,
-                                  float2* __restrict__ cs, int T, int n_freq) {
+                                  float2* __restrict__ cs, int T, int n_freq, float mag) {
   pdl_launch();
   pdl_wait();
   const int idx = blockIdx.x * blockDim.x + threadIdx.x;
@@ -247,14 +247,14 @@ __global__ void rope_table_kernel(const int* __restrict__ positions, const float
   const int t = idx / n_freq, i = idx % n_freq;
   float sn, c;
   sincosf((float)positions[t] * inv_freq[i], &sn, &c);
-  cs[idx] = make_float2(c, sn);
+  cs[idx] = make_float2(c * mag, sn * mag);
 }
-RLLM_API int rllm_rope_table(const int* positions, const float* inv_freq, void* cs, int T, int n_freq,
+RLLM_API int rllm_rope_table(const int* positions, const float* inv_freq, void* cs, int T, int n_freq, float mag,
                              void* stream) {
   if (T <= 0 || n_freq <= 0) return 0;
   const int n = T * n_freq;
   return launch_ex(rope_table_kernel, dim3((n + 255) / 256), dim3(256), 0, (cudaStream_t)stream, 1, positions,
-                   inv_freq, (float2*)cs, T, n_freq);
+                   inv_freq, (float2*)cs, T, n_freq, mag);
 }
 
 template <typename T>

@@ -72,6 +72,7 @@ struct Args {
   int splits; float* pacc; float* pml;
   int page_shift;              // log2(page_size), or -1 when it is no power of two
   int keep_first;              // positions below this number are seen whatever the window says
+  SoftCap cap;                 // cap.c > 0: scores are bounded, cap tanh(score / cap)
 };
 
 __device__ __forceinline__ int first_key(int pos, int window, int chunk) {
@@ -206,6 +207,7 @@ __global__ void __launch_bounds__(THREADS) sink_attention_mma_kernel(const Args 
     m1 = v1 ? 0.f : -INFINITY;
   }
 
+  const float sl = p.cap.c > 0.f ? 1.f : p.scale_log2;
   // STAGES - 1 tiles are on their way while one is worked on (a commit per tile, empty past the end, so that
   // the count of groups in flight says which tile has landed)
 #pragma unroll
@@ -240,6 +242,14 @@ __global__ void __launch_bounds__(THREADS) sink_attention_mma_kernel(const Args 
         }
       }
     }
+    // a bounded score leaves the bound in the log2 domain, where it needs no further scale
+    if (p.cap.c > 0.f) {
+#pragma unroll
+      for (int nt = 0; nt < NT; ++nt) {
+        sc[nt][0] = softcap_log2(sc[nt][0], p.cap); sc[nt][1] = softcap_log2(sc[nt][1], p.cap);
+        sc[nt][2] = softcap_log2(sc[nt][2], p.cap); sc[nt][3] = softcap_log2(sc[nt][3], p.cap);
+      }
+    }
     // mask (only where a row's edge crosses the tile), scale into the log2 domain, running maximum
     const int key0 = tile * KEYS + kofs;
     float mx0 = -INFINITY, mx1 = -INFINITY;
@@ -251,8 +261,8 @@ __global__ void __launch_bounds__(THREADS) sink_attention_mma_kernel(const Args 
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
           const int j = key0 + nt * 8 + (lane & 3) * 2 + e;
-          const float a = (v0 && (j >= st0 || j < p.keep_first) && j <= pos0) ? sc[nt][e] * p.scale_log2 : -INFINITY;
-          const float c = (v1 && (j >= st1 || j < p.keep_first) && j <= pos1) ? sc[nt][2 + e] * p.scale_log2 : -INFINITY;
+          const float a = (v0 && (j >= st0 || j < p.keep_first) && j <= pos0) ? sc[nt][e] * sl : -INFINITY;
+          const float c = (v1 && (j >= st1 || j < p.keep_first) && j <= pos1) ? sc[nt][2 + e] * sl : -INFINITY;
           sc[nt][e] = a; sc[nt][2 + e] = c;
           mx0 = fmaxf(mx0, a); mx1 = fmaxf(mx1, c);
         }
@@ -261,7 +271,7 @@ __global__ void __launch_bounds__(THREADS) sink_attention_mma_kernel(const Args 
 #pragma unroll
       for (int nt = 0; nt < NT; ++nt) {
 #pragma unroll
-        for (int e = 0; e < 4; ++e) sc[nt][e] *= p.scale_log2;
+        for (int e = 0; e < 4; ++e) sc[nt][e] *= sl;
         mx0 = fmaxf(mx0, fmaxf(sc[nt][0], sc[nt][1])); mx1 = fmaxf(mx1, fmaxf(sc[nt][2], sc[nt][3]));
       }
     }
@@ -438,7 +448,7 @@ RLLM_API int rllm_sink_attention_mma(const void* q, long long q_stride, const vo
                                      int bt_stride, int num_seqs, int n_tokens, int max_q_len, int nh, int nkv, int kd, int vd,
                                      int page_size, float scale, int window, int chunk, const float* sinks, const float* gate,
                                      int gate_ld, int splits, float* pacc, float* pml, int keep_first, int sigmoid,
-                                     void* stream) {
+                                     float softcap, void* stream) {
   using namespace sinkmma;
   if (n_tokens <= 0 || num_seqs <= 0) return 0;
   if (!rllm_sink_attention_mma_supported(DT_BF16, kd, vd, page_size) || nkv <= 0 || nh % nkv || splits < 1 || splits > 64 ||
@@ -450,7 +460,7 @@ RLLM_API int rllm_sink_attention_mma(const void* q, long long q_stride, const vo
   if (tiles > 2147483647LL || nkv > 65535) return ERR_TOO_LARGE;
   Args a = {(const bf16*)q, q_stride, (const bf16*)kcache, (const bf16*)vcache, (bf16*)out, out_stride, positions, cu_q,
             block_table, bt_stride, num_seqs, nh, nkv, kd, vd, page_size, scale * 1.4426950408889634f, window, chunk, sinks,
-            gate, gate_ld, splits, pacc, pml, -1, keep_first};
+            gate, gate_ld, splits, pacc, pml, -1, keep_first, make_softcap(softcap, scale)};
   for (int sft = 0; sft < 31; ++sft) if ((1 << sft) == page_size) a.page_shift = sft;
   cudaStream_t s = (cudaStream_t)stream;
   const dim3 grid((unsigned)tiles, (unsigned)nkv, (unsigned)splits);

@@ -4,6 +4,8 @@
 // postnorm:  s = alpha * h[t] + sum over p of y[t, p, :] (+ sigmoid(zg[t]) * y2[t]);  h[t] = w * s / sqrt(mean(s^2) + eps),
 //            float throughout, the parts added in order. Also writes h[t] in the run's storage type (`copy`),
 //            which is what the next sublayer's products read.
+// output_norm: the same operands with the norm on the sublayer's output alone: s = sum over p of y[t, p, :] (+ the gated
+//            y2); h[t] += alpha * w * s / sqrt(mean(s^2) + eps); `copy` as above.
 // cast_rows: the stream in the run's storage type (the first layer's input).
 // gated_act: out[r, i] = act(scale_r * g) * (scale_r * u) for gu [R, 2F] (float or storage type), act = silu; the
 //            columns of gu come in blocks of `block` gate columns followed by their up columns (block = F: all gate
@@ -13,7 +15,8 @@ using namespace rllm;
 
 namespace {
 
-template <typename TO>
+// OUT: the norm is on the sublayer's output alone (output_norm).
+template <typename TO, bool OUT>
 __global__ void postnorm_kernel(float* __restrict__ h, const float* __restrict__ y, int parts, const float* __restrict__ y2,
                                 const float* __restrict__ zg, int zg_ld, float alpha, const float* __restrict__ w, int H,
                                 float eps, TO* __restrict__ copy) {
@@ -28,7 +31,7 @@ __global__ void postnorm_kernel(float* __restrict__ h, const float* __restrict__
   const float g2 = (y2 && zg) ? 1.f / (1.f + expf(-zg[t * zg_ld])) : 1.f;
   float ss = 0.f;
   for (int i = threadIdx.x; i < H; i += blockDim.x) {
-    float v = alpha * hr[i];
+    float v = OUT ? 0.f : alpha * hr[i];
     if (yr)
       for (int p = 0; p < parts; ++p) v += yr[(size_t)p * H + i];
     if (y2r) v = fmaf(g2, y2r[i], v);
@@ -38,7 +41,8 @@ __global__ void postnorm_kernel(float* __restrict__ h, const float* __restrict__
   ss = block_sum(ss, red);
   const float r = 1.f / sqrtf(ss / (float)H + eps);
   for (int i = threadIdx.x; i < H; i += blockDim.x) {
-    const float v = row[i] * r * w[i];
+    const float n = row[i] * r * w[i];
+    const float v = OUT ? fmaf(alpha, n, hr[i]) : n;
     hr[i] = v;
     if (copy) copy[t * H + i] = from_f32<TO>(v);
   }
@@ -46,7 +50,7 @@ __global__ void postnorm_kernel(float* __restrict__ h, const float* __restrict__
 
 // The same for rows of 4 * VPT * blockDim numbers at most: every thread keeps VPT float4 of the row in registers,
 // all of a row's loads are in flight together (a step of single tokens is a handful of rows: latency is all).
-template <typename TO, int VPT>
+template <typename TO, int VPT, bool OUT>
 __global__ void __launch_bounds__(1024) postnorm_vec_kernel(float* __restrict__ h, const float* __restrict__ y, int parts,
                                                            const float* __restrict__ y2, const float* __restrict__ zg,
                                                            int zg_ld, float alpha, const float* __restrict__ w, int H,
@@ -59,7 +63,7 @@ __global__ void __launch_bounds__(1024) postnorm_vec_kernel(float* __restrict__ 
   float4* hr = reinterpret_cast<float4*>(h + t * H);
   const float4* yr = y ? reinterpret_cast<const float4*>(y + t * parts * H) : nullptr;
   const float4* y2r = y2 ? reinterpret_cast<const float4*>(y2 + t * H) : nullptr;
-  float4 v[VPT], e[VPT];
+  float4 v[VPT], e[VPT], x[OUT ? VPT : 1];
 #pragma unroll
   for (int k = 0; k < VPT; ++k) {
     const int i = threadIdx.x + k * blockDim.x;
@@ -68,7 +72,10 @@ __global__ void __launch_bounds__(1024) postnorm_vec_kernel(float* __restrict__ 
   }
   const float g2 = (y2 && zg) ? 1.f / (1.f + expf(-zg[t * zg_ld])) : 1.f;
 #pragma unroll
-  for (int k = 0; k < VPT; ++k) { v[k].x *= alpha; v[k].y *= alpha; v[k].z *= alpha; v[k].w *= alpha; }
+  for (int k = 0; k < VPT; ++k) {
+    if (OUT) { x[OUT ? k : 0] = v[k]; v[k] = make_float4(0.f, 0.f, 0.f, 0.f); }
+    else { v[k].x *= alpha; v[k].y *= alpha; v[k].z *= alpha; v[k].w *= alpha; }
+  }
   if (yr) {
     for (int p = 0; p < parts; ++p) {
 #pragma unroll
@@ -91,7 +98,11 @@ __global__ void __launch_bounds__(1024) postnorm_vec_kernel(float* __restrict__ 
     const int i = threadIdx.x + k * blockDim.x;
     if (i < n4) {
       const float4 ww = reinterpret_cast<const float4*>(w)[i];
-      const float4 o = make_float4(v[k].x * r * ww.x, v[k].y * r * ww.y, v[k].z * r * ww.z, v[k].w * r * ww.w);
+      float4 o = make_float4(v[k].x * r * ww.x, v[k].y * r * ww.y, v[k].z * r * ww.z, v[k].w * r * ww.w);
+      if (OUT) {
+        const float4 b = x[OUT ? k : 0];
+        o = make_float4(fmaf(alpha, o.x, b.x), fmaf(alpha, o.y, b.y), fmaf(alpha, o.z, b.z), fmaf(alpha, o.w, b.w));
+      }
       hr[i] = o;
       if (copy) {
         TO* c = copy + t * H + 4 * (size_t)i;
@@ -101,7 +112,7 @@ __global__ void __launch_bounds__(1024) postnorm_vec_kernel(float* __restrict__ 
   }
 }
 
-template <typename TO>
+template <typename TO, bool OUT>
 int launch_postnorm(float* h, const float* y, int parts, const float* y2, const float* zg, int zg_ld, float alpha,
                     const float* w, int T, int H, float eps, TO* copy, cudaStream_t s) {
   const bool vec = H % 4 == 0 && !((uintptr_t)h & 15) && !((uintptr_t)y & 15) && !((uintptr_t)y2 & 15) && !((uintptr_t)w & 15);
@@ -109,16 +120,16 @@ int launch_postnorm(float* h, const float* y, int parts, const float* y2, const 
     const int n4 = H / 4;
     if (n4 <= 1024) {
       const int threads = (n4 + 31) / 32 * 32;
-      return launch_ex(postnorm_vec_kernel<TO, 1>, dim3(T), dim3(threads), 0, s, 1, h, y, parts, y2, zg, zg_ld, alpha, w, H, eps, copy);
+      return launch_ex(postnorm_vec_kernel<TO, 1, OUT>, dim3(T), dim3(threads), 0, s, 1, h, y, parts, y2, zg, zg_ld, alpha, w, H, eps, copy);
     }
     const int threads = ((n4 + 3) / 4 + 31) / 32 * 32;
-    return launch_ex(postnorm_vec_kernel<TO, 4>, dim3(T), dim3(threads), 0, s, 1, h, y, parts, y2, zg, zg_ld, alpha, w, H, eps, copy);
+    return launch_ex(postnorm_vec_kernel<TO, 4, OUT>, dim3(T), dim3(threads), 0, s, 1, h, y, parts, y2, zg, zg_ld, alpha, w, H, eps, copy);
   }
   static bool done[64] = {};
   const int smem = H * (int)sizeof(float);
-  if (smem > 48 * 1024) { const int rc = allow_dynamic_smem(postnorm_kernel<TO>, smem, done); if (rc) return rc; }
+  if (smem > 48 * 1024) { const int rc = allow_dynamic_smem(postnorm_kernel<TO, OUT>, smem, done); if (rc) return rc; }
   const int threads = H >= 1024 ? 256 : (H >= 256 ? 128 : 64);
-  return launch_ex(postnorm_kernel<TO>, dim3(T), dim3(threads), (size_t)smem, s, 1, h, y, parts, y2, zg, zg_ld, alpha, w, H, eps, copy);
+  return launch_ex(postnorm_kernel<TO, OUT>, dim3(T), dim3(threads), (size_t)smem, s, 1, h, y, parts, y2, zg, zg_ld, alpha, w, H, eps, copy);
 }
 
 __global__ void cast_rows_kernel(const float* __restrict__ x, bf16* __restrict__ out, long long n) {
@@ -175,15 +186,18 @@ inline int blocks_for(long long n) { return (int)((n + 255) / 256 < 2368 ? (n + 
 
 // h [T, H] float in place; y [T, parts, H] float or null; y2 [T, H] float or null with zg (logits, one per row at
 // stride zg_ld) or null; copy [T, H] of type copy_dt or null.
+// output != 0: output_norm (alpha the coefficient of the normed output).
 RLLM_API int rllm_postnorm(float* h, const float* y, int parts, const float* y2, const float* zg, int zg_ld, float alpha,
-                           const float* w, int T, int H, float eps, void* copy, int copy_dt, void* stream) {
+                           const float* w, int T, int H, float eps, void* copy, int copy_dt, int output, void* stream) {
   if (T <= 0) return 0;
   if (H <= 0 || parts < 0 || (size_t)H * sizeof(float) > 200 * 1024) return ERR_BAD_SIZE;
   cudaStream_t s = (cudaStream_t)stream;
   if (copy && copy_dt == DT_BF16)
-    return launch_postnorm<bf16>(h, y, parts, y2, zg, zg_ld, alpha, w, T, H, eps, (bf16*)copy, s);
+    return output ? launch_postnorm<bf16, true>(h, y, parts, y2, zg, zg_ld, alpha, w, T, H, eps, (bf16*)copy, s)
+                  : launch_postnorm<bf16, false>(h, y, parts, y2, zg, zg_ld, alpha, w, T, H, eps, (bf16*)copy, s);
   if (copy && copy_dt != DT_F32) return ERR_BAD_DTYPE;
-  return launch_postnorm<float>(h, y, parts, y2, zg, zg_ld, alpha, w, T, H, eps, (float*)copy, s);
+  return output ? launch_postnorm<float, true>(h, y, parts, y2, zg, zg_ld, alpha, w, T, H, eps, (float*)copy, s)
+                : launch_postnorm<float, false>(h, y, parts, y2, zg, zg_ld, alpha, w, T, H, eps, (float*)copy, s);
 }
 
 RLLM_API int rllm_cast_rows(const float* x, void* out, long long n, void* stream) {

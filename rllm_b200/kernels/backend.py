@@ -130,16 +130,16 @@ class Backend:
         return ops.gemm_simt(x, w_gate_up, ops.EPI_SWIGLU)
 
     # ---- position encoding + cache write, attention
-    def rope_table(self, ctx, positions, inv_freq, rot_dim, key=None):
+    def rope_table(self, ctx, positions, inv_freq, rot_dim, key=None, mag=1.0):
         """The step's (cos, sin) table for one rotation rule, made at its first use in a forward
-        pass and shared by the layers with the same rule (`key`)."""
+        pass and shared by the layers with the same rule (`key`). `mag`: a factor on both."""
         if ctx is None:
             return None
         tables = ctx.per_forward.setdefault("rope_tables", {})
         key = key if key is not None else (inv_freq.data_ptr(), rot_dim)
         t = tables.get(key)
         if t is None:
-            t = tables[key] = ops.rope_table(positions, inv_freq[: rot_dim // 2].contiguous(), ctx.num_tokens)
+            t = tables[key] = ops.rope_table(positions, inv_freq[: rot_dim // 2].contiguous(), ctx.num_tokens, mag)
         return t
 
     def qkv_rope_cache_write(self, x, w_qkv, bias, positions, inv_freq, cache, nh, nkv, hd, rot_dim=None,
@@ -276,10 +276,18 @@ class Backend:
         self._sink.postnorm(h, parts, alpha, w, eps, extra, gate, copy)
         return h if copy is None else copy
 
+    def output_norm(self, h, y, coef, w, eps):
+        """h += coef * w * y / rms(y), in float and in place; y as for `postnorm`. Returns the new stream in the run's
+        storage type (h itself in the 32-bit run)."""
+        parts, extra, gate = (y.parts, y.extra, y.extra_gate) if hasattr(y, "parts") else (y, None, None)
+        copy = None if self.dtype == torch.float32 else torch.empty(h.shape, dtype=self.dtype, device=h.device)
+        self._sink.postnorm(h, parts, coef, w, eps, extra, gate, copy, output=True)
+        return h if copy is None else copy
+
     def linear_act(self, x, w, act):
-        """act(x W^T) in the run dtype; act "relu2" = max(., 0)^2, "gelu_tanh" = gelu in its tanh form (on the float
-        product, rounded once)."""
-        if act not in ("relu2", "gelu_tanh"):
+        """act(x W^T) in the run dtype; act "relu2" = max(., 0)^2, "gelu_tanh" = gelu in its tanh form, "gelu_erf" in its
+        erf form (on the float product, rounded once)."""
+        if act not in ("relu2", "gelu_tanh", "gelu_erf"):
             raise ops.KernelError(f"activation {act!r} has no kernel")
         fuse = os.environ.get("RLLM_B200_NO_ACT_FUSION") != "1"
         if fuse and self._fused_norm(x, w):                                  # the norm in front, the activation behind
@@ -287,6 +295,8 @@ class Backend:
         x = x.tensor() if isinstance(x, Normed) else x
         if self._tc(x, w) and fuse:
             return self._sm100.gemm(x, w, ops.EPI_STORE, act=act)            # in the product's store epilogue
+        if act == "gelu_erf":
+            return ops.gemm_simt(x, w, ops.EPI_GELU_ERF)
         if act == "gelu_tanh":
             return self._hy.act_rows(self.linear_f32(x, w, tag="up"), self.dtype, act)
         if self._tc(x, w):
@@ -294,18 +304,22 @@ class Backend:
         return ops.gemm_simt(x, w, ops.EPI_RELU2)
 
     def qk_norm_rope_store(self, proj, q_off, k_off, v_off, nh, nkv, kd, vd, rot, wq, wk, eps, table, cache, vfirst=None,
-                           lam=None):
-        """`vfirst`, `lam`: the values are cached as (1 - lam) v + lam vfirst (another layer's values of the same tokens)."""
+                           lam=None, row_norm=False, interleaved=False):
+        """`vfirst`, `lam`: the values are cached as (1 - lam) v + lam vfirst (another layer's values of the same tokens).
+        `row_norm`: queries and keys are normed over all heads together; `interleaved`: rotation pairs (2i, 2i + 1)."""
         writes = cache.writes
         self._sink.qk_norm_rope_store(proj, q_off, k_off, v_off, nh, nkv, kd, vd, rot, wq, wk, eps, table,
                                       cache.slots if writes else None, cache.k if writes else None,
-                                      cache.v if writes else None, vfirst if writes else None, lam if writes else None)
+                                      cache.v if writes else None, vfirst if writes else None, lam if writes else None, row_norm,
+                                      interleaved)
 
-    def sink_attention(self, q, cache, ctx, nh, scale, window, chunk, sinks, gate, keep_first=0, sigmoid=False):
+    def sink_attention(self, q, cache, ctx, nh, scale, window, chunk, sinks, gate, keep_first=0, sigmoid=False,
+                       softcap=None):
         """Attention with a window and/or block mask, a sink and an output gate over pages whose keys and values
         may differ in size: bfloat16 on the tensor cores where the kernel takes the sizes, else (and in the
         32-bit run) in float on the CUDA cores. `keep_first`: positions below it are seen whatever the window says.
-        `sigmoid`: no softmax, a visible key's weight is sigmoid(score + sinks[head])."""
+        `sigmoid`: no softmax, a visible key's weight is sigmoid(score + sinks[head]). `softcap`: scores bounded,
+        softcap * tanh(score / softcap)."""
         sk = self._sink
         kd, vd, nkv = cache.k.shape[3], cache.v.shape[3], cache.k.shape[1]
         tc = self.fast and os.environ.get("RLLM_B200_NO_TC_ATTENTION") != "1"
@@ -316,20 +330,20 @@ class Backend:
         if chunk:
             keys = min(keys, chunk)
         G = nh // nkv
-        if tc and kd == vd and self._sm100.attention_supported(q, cache.k):
+        if tc and kd == vd and scale > 0 and self._sm100.attention_supported(q, cache.k):
             # equal head sizes of 64 or 128: the kernels of plain grouped-query attention take the mask, the sink
             # and the gate as well (the clusters of the decode kernel, tcgen05 for long portions); kept first keys and
             # sigmoid weights only the tcgen05 kernel does
             sm = self._sm100
             if ctx.max_q_len == 1 and not keep_first and not sigmoid and sm.decode_supported(q, cache.k, nh):
                 return sm.attention_decode(q, cache.k, cache.v, ctx.kv_lens, cache.block_table, nh, scale, window, keys,
-                                           chunk=chunk, sinks=sinks, gate=gate)
+                                           chunk=chunk, sinks=sinks, gate=gate, softcap=softcap)
             lens = ctx.q_lens_host
             if ctx.max_q_len * G >= 128 and ctx.max_kv_len >= sm.TC_ATTENTION_MIN_KEYS and sm.prefill_tc_supported(q, cache.k) \
                     and lens is not None and min(lens) * G >= 128:
                 return sm.attention_prefill_tc(q, cache.k, cache.v, ctx.cu_q, ctx.kv_lens, cache.block_table, ctx.max_q_len,
                                                nh, scale, window, chunk=chunk, sinks=sinks, gate=gate, keep_first=keep_first,
-                                               sigmoid=sigmoid)
+                                               sigmoid=sigmoid, softcap=softcap)
         if tc and sk.mma_supported(q.dtype, kd, vd, cache.page_size):
             tiles = 0
             for ql in (ctx.q_lens_host if not ctx.graph_safe else [1] * ctx.num_seqs):
@@ -339,9 +353,9 @@ class Backend:
             splits = max(1, min(16, 4 * self.sm_count // max(tiles, 1), keys // 128))
             return sk.sink_attention_mma(q, cache.k, cache.v, ctx.token_seq, ctx.positions, cache.block_table, ctx.cu_q,
                                          ctx.num_seqs, ctx.max_q_len, nh, scale, window, chunk, sinks, gate, splits, keys,
-                                         keep_first, sigmoid)
+                                         keep_first, sigmoid, softcap)
         return sk.sink_attention_simt(q, cache.k, cache.v, ctx.token_seq, ctx.positions, cache.block_table, nh, scale,
-                                      window, chunk, sinks, gate, keep_first, sigmoid)
+                                      window, chunk, sinks, gate, keep_first, sigmoid, softcap)
 
     def latent_prepare(self, *a, **k):
         return self._mix.latent_prepare(*a, **k)
@@ -372,7 +386,7 @@ class Backend:
         return self._mix.gla_finish(*a, **k)
 
     # ---- recurrent mixers with a short convolution, attention with mixed heads, layers whose sublayers run side by
-    # side (library "hybrid")
+    # side (libraries "recurrent" and "hybrid")
     @property
     def _hy(self):
         from . import hybrid

@@ -1,5 +1,5 @@
-"""Python face of the library "hybrid": recurrent mixers over a per-request state with a short causal
-convolution in front (csrc/recurrent.cu), grouped-query attention whose heads' softmax weights are mixed by a
+"""Python face of the libraries "recurrent" (recurrent mixers over a per-request state with a short causal
+convolution in front, csrc/recurrent.cu) and "hybrid": grouped-query attention whose heads' softmax weights are mixed by a
 matrix (csrc/talk_attention.cu), and the row-wise work of layers whose sublayers run side by side on one normed
 input (csrc/row_mix.cu). Every function checks shapes, dtypes and devices and then calls an `extern "C"`
 launcher on torch's current stream; there is no CPU or library path behind them.
@@ -15,12 +15,7 @@ from .ops import KernelError, _check, _cuda, _dt, _fn, _ptr, _stream
 
 _P, _LL = ops._P, c_longlong
 
-ops.register_signatures("hybrid", {
-    "rllm_pair_embed": [_P, _P, _P, _P, _P, _P, _P, _P, c_int, _P, c_float, _P, c_int, c_int, c_int, c_int, c_int, _LL, _LL,
-                        _P, _P],
-    "rllm_combine": [_P, _P, _P, _P, _P, c_float, c_float, _P, c_int, _P, c_int, _P, c_int, c_int, c_int, _P],
-    "rllm_glu_act": [_P, c_int, _LL, _P, c_int, c_int, c_int, c_int, c_float, c_float, c_int, _P],
-    "rllm_add_bias_f32": [_P, _P, c_int, c_int, _P],
+ops.register_signatures("recurrent", {
     "rllm_short_conv": [c_int, _P, _LL, c_int, c_int, c_int, _P, _P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, _P],
     "rllm_unit_heads": [_P, _LL, c_int, c_int, c_int, c_float, c_float, c_int, _P],
     "rllm_softplus_decay": [c_int, _P, _LL, c_int, _P, _P, c_int, c_int, c_int, _P, _P, _P],
@@ -28,6 +23,13 @@ ops.register_signatures("hybrid", {
     "rllm_state_scan": [c_int, _P, _LL, c_int, _P, _LL, c_int, _P, _LL, _P, c_int, _P, _LL, _P, _P, c_int, c_int, c_int,
                         c_int, _P, _P, _P, _P, c_int, _P],
     "rllm_gated_norm": [_P, _P, c_int, _LL, _P, c_int, c_float, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P],
+})
+ops.register_signatures("hybrid", {
+    "rllm_pair_embed": [_P, _P, _P, _P, _P, _P, _P, _P, c_int, _P, c_float, _P, c_int, c_int, c_int, c_int, c_int, _LL, _LL,
+                        _P, _P],
+    "rllm_combine": [_P, _P, _P, _P, _P, c_float, c_float, _P, c_int, _P, c_int, _P, c_int, c_int, c_int, _P],
+    "rllm_glu_act": [_P, c_int, _LL, _P, c_int, c_int, c_int, c_int, c_float, c_float, c_int, _P],
+    "rllm_add_bias_f32": [_P, _P, c_int, c_int, _P],
     "rllm_value_norm_store": [c_int, _P, _LL, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, _P, _P, _P, c_int, _P],
     "rllm_talk_attention_simt": [c_int, _P, _LL, _P, _P, _P, _P, _P, _LL, _P, _P, _P, c_int, c_int, c_int, c_int, c_int,
                                  c_int, c_float, c_int, c_int, _P],
@@ -245,7 +247,7 @@ def short_conv(x, col0, channels, w, bias, token_seq, positions, cu_q, num_seqs,
             raise KernelError(f"the convolution tail must be [slots, {taps - 1}, {channels}], got {list(tail.shape)}")
     out = torch.empty((T, channels), dtype=torch.float32, device=x.device)
     keeps = state_slots is not None and taps > 1
-    _check(_fn("hybrid", "rllm_short_conv")(
+    _check(_fn("recurrent", "rllm_short_conv")(
         _dt(x, "x"), x.data_ptr(), x.stride(0), int(col0), int(channels), taps, w.data_ptr(), _ptr(bias), token_seq.data_ptr(),
         positions.data_ptr(), cu_q.data_ptr(), _ptr(state_slots), _ptr(tail) if state_slots is not None else None,
         out.data_ptr(), T, int(num_seqs), int(bool(silu)), _stream()), "short_conv", 2 if keeps else 1)
@@ -259,7 +261,7 @@ def unit_heads(x, col0, heads, dim, scale=1.0, eps=1e-6) -> torch.Tensor:
     if x.dtype != torch.float32:
         raise KernelError("unit_heads works on float32 rows")
     _rows(x, "x", col0 + heads * dim)
-    _check(_fn("hybrid", "rllm_unit_heads")(x.data_ptr(), x.stride(0), int(col0), int(heads), int(dim), float(scale), float(eps),
+    _check(_fn("recurrent", "rllm_unit_heads")(x.data_ptr(), x.stride(0), int(col0), int(heads), int(dim), float(scale), float(eps),
                                             x.shape[0], _stream()), "unit_heads")
     return x
 
@@ -276,7 +278,7 @@ def softplus_decay(z, col0, n, bias, a_log, want_step=False):
     T = z.shape[0]
     step = torch.empty((T, n), dtype=torch.float32, device=z.device) if want_step else None
     decay = torch.empty((T, n), dtype=torch.float32, device=z.device)
-    _check(_fn("hybrid", "rllm_softplus_decay")(_dt(z, "z"), z.data_ptr(), z.stride(0), int(col0), _ptr(bias), a_log.data_ptr(), T,
+    _check(_fn("recurrent", "rllm_softplus_decay")(_dt(z, "z"), z.data_ptr(), z.stride(0), int(col0), _ptr(bias), a_log.data_ptr(), T,
                                                 int(n), n // a_log.numel(), _ptr(step), decay.data_ptr(), _stream()),
            "softplus_decay")
     return step, decay
@@ -311,7 +313,7 @@ def state_scan(q, q_heads, k, k_heads, v, decay, heads, dim, vdim, cu_q, num_seq
     if skip is not None:
         _f32(skip, "skip", (heads,))
     out = torch.empty((T, heads, vdim), dtype=torch.float32, device=q.device)
-    _check(_fn("hybrid", "rllm_state_scan")(
+    _check(_fn("recurrent", "rllm_state_scan")(
         _dt(beta, "beta") if beta is not None else 0, q.data_ptr(), q.stride(0), int(q_heads), k.data_ptr(), k.stride(0),
         int(k_heads), v.data_ptr(), v.stride(0), decay.data_ptr(), int(per_channel), _ptr(beta),
         beta.stride(0) if beta is not None else 0, _ptr(vscale), _ptr(skip), int(num_seqs), int(heads), int(dim), int(vdim),
@@ -337,7 +339,7 @@ def gated_norm(y, gate, gate_col0, weight, eps, groups, out_dtype, gate_first: b
         _rows(gate, "gate", gate_col0 + n)
         g = gate.data_ptr() + gate_col0 * gate.element_size()
     out = torch.empty((T, n), dtype=out_dtype, device=y.device)
-    _check(_fn("hybrid", "rllm_gated_norm")(y.data_ptr(), g, _dt(gate, "gate") if gate is not None else 0,
+    _check(_fn("recurrent", "rllm_gated_norm")(y.data_ptr(), g, _dt(gate, "gate") if gate is not None else 0,
                                             gate.stride(0) if gate is not None else 0, weight.data_ptr(), weight.numel(),
                                             float(eps), out.data_ptr(), _dt(out, "out"), T, int(groups), n // groups,
                                             int(bool(gate_first)), GATE_ACTS[act], _stream()), "gated_norm")

@@ -18,6 +18,7 @@ _DT = {torch.float32: DT_F32, torch.bfloat16: DT_BF16}
 
 EPI_STORE, EPI_STORE_F32, EPI_ACCUM_F32, EPI_SWIGLU = 0, 1, 2, 3
 EPI_RELU2 = 4          # the CUDA-core product only: max(., 0)^2 of the float result, stored in the operand type
+EPI_GELU_ERF = 5       # likewise: gelu(.) in its erf form
 
 _ERR = {-1: "unsupported dtype", -2: "unsupported size", -3: "misaligned operand",
         -4: "problem too large for this kernel", -5: "kernel set-up failed"}
@@ -32,7 +33,7 @@ _SIGS = {
     "simt": {
         "rllm_embed": [_P, _P, c_int, _P, c_int, c_int, c_int, _P, c_float, _P],
         "rllm_rmsnorm": [_P, _P, _P, c_int, _P, c_int, c_int, c_int, c_float, _P],
-        "rllm_rope_table": [_P, _P, _P, c_int, c_int, _P],
+        "rllm_rope_table": [_P, _P, _P, c_int, c_int, c_float, _P],
         "rllm_rope_cache_write": [_P, c_int, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int,
                                   c_int, _P],
         "rllm_gather_rows": [_P, _P, _P, c_int, c_int, _P],
@@ -150,8 +151,8 @@ def rmsnorm(x: torch.Tensor, w: torch.Tensor, eps: float, out_dtype: torch.dtype
     return out
 
 
-def rope_table(positions: torch.Tensor, inv_freq: torch.Tensor, T: int) -> torch.Tensor:
-    """(cos, sin)(positions[t] * inv_freq[i]) as float32 [T, len(inv_freq), 2]: a step's rotations,
+def rope_table(positions: torch.Tensor, inv_freq: torch.Tensor, T: int, mag: float = 1.0) -> torch.Tensor:
+    """mag * (cos, sin)(positions[t] * inv_freq[i]) as float32 [T, len(inv_freq), 2]: a step's rotations,
     made once and read by every layer."""
     _cuda(positions, "positions"); _cuda(inv_freq, "inv_freq")
     if positions.dtype != torch.int32 or positions.numel() < T or inv_freq.dtype != torch.float32 \
@@ -159,7 +160,7 @@ def rope_table(positions: torch.Tensor, inv_freq: torch.Tensor, T: int) -> torch
         raise KernelError("rope_table takes int32 positions [T] and float32 inverse frequencies")
     out = torch.empty((T, inv_freq.numel(), 2), dtype=torch.float32, device=positions.device)
     _check(_fn("simt", "rllm_rope_table")(positions.data_ptr(), inv_freq.data_ptr(), out.data_ptr(), T,
-                                          inv_freq.numel(), _stream()), "rope_table")
+                                          inv_freq.numel(), float(mag), _stream()), "rope_table")
     return out
 
 
@@ -250,7 +251,7 @@ def silu_gate(gu: torch.Tensor) -> torch.Tensor:
 def gemm_simt(a: torch.Tensor, w: torch.Tensor, epilogue: int, out: torch.Tensor | None = None,
               bias: torch.Tensor | None = None) -> torch.Tensor:
     """C = A W^T on the CUDA cores (float accumulate). a [T, K]; w [N, K] ([2N, K] for SwiGLU). Epilogue
-    EPI_RELU2 stores max(C, 0)^2 in a's dtype."""
+    EPI_RELU2 stores max(C, 0)^2 in a's dtype, EPI_GELU_ERF gelu(C) in its erf form."""
     _cuda(a, "a"); _cuda(w, "w")
     if a.dim() != 2 or w.dim() != 2 or a.stride(1) != 1 or not w.is_contiguous():
         raise KernelError("gemm takes a [T, K] (unit inner stride) and a contiguous w [N, K]")

@@ -181,13 +181,18 @@ class OpProfile:
         parts = y.parts if hasattr(y, "parts") else y
         return self._timed("add+norm", _nbytes(parts, getattr(y, "extra", None)) + 10 * h.numel(), 0, self._be.postnorm, h, y, *a, **k)
 
+    def output_norm(self, h, y, *a, **k):
+        parts = y.parts if hasattr(y, "parts") else y
+        return self._timed("norm+add", _nbytes(parts, getattr(y, "extra", None)) + 10 * h.numel(), 0, self._be.output_norm, h, y,
+                           *a, **k)
+
     def linear_act(self, x, w, act):
         return self._product("up", x, w, self._be.linear_act, x, w, act)
 
     def qk_norm_rope_store(self, proj, *a, **k):
         return self._timed("qk_norm+rope", 2 * _nbytes(proj), 0, self._be.qk_norm_rope_store, proj, *a, **k)
 
-    def sink_attention(self, q, cache, ctx, nh, scale, window, chunk, sinks, gate, keep_first=0, sigmoid=False):
+    def sink_attention(self, q, cache, ctx, nh, scale, window, chunk, sinks, gate, keep_first=0, sigmoid=False, softcap=None):
         kd, vd, nkv = cache.k.shape[3], cache.v.shape[3], cache.k.shape[1]
         lens, qs = ctx.kv_lens_host, ctx.q_lens_host
         if lens is None:
@@ -204,7 +209,7 @@ class OpProfile:
             seen_keys += n - first + min(keep_first, first)
         nbytes = seen_keys * nkv * (kd + vd) * cache.k.element_size() + _nbytes(q) + q.shape[0] * nh * vd * q.element_size()
         return self._timed("sigmoid_attention" if sigmoid else "attention", nbytes, 2 * nh * (kd + vd) * pairs,
-                           self._be.sink_attention, q, cache, ctx, nh, scale, window, chunk, sinks, gate, keep_first, sigmoid)
+                           self._be.sink_attention, q, cache, ctx, nh, scale, window, chunk, sinks, gate, keep_first, sigmoid, softcap)
 
     def latent_prepare(self, proj, *a, **k):
         return self._timed("latent_prepare", 2 * _nbytes(proj), 0, self._be.latent_prepare, proj, *a, **k)

@@ -1,5 +1,5 @@
-"""Python face of the library "sink": grouped-query attention with a per-head norm of queries and keys,
-a rotation of part of a head, keys and values of different sizes, a window and/or block mask, a sink in
+"""Python face of the library "sink": grouped-query attention with a norm of queries and keys (per head or over all
+heads together), a rotation of part of a head, keys and values of different sizes, a window and/or block mask, a sink in
 the softmax and an output gate (csrc/sink_attention.cu), and the row-wise work of layers that norm after
 the sum (csrc/stream_ops.cu). Every function checks shapes, dtypes and devices and then calls an
 `extern "C"` launcher on torch's current stream; there is no CPU or library path behind them.
@@ -17,13 +17,13 @@ _P, _LL = ops._P, c_longlong
 
 ops.register_signatures("sink", {
     "rllm_qk_norm_rope_store": [c_int, _P, _LL, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P,
-                                c_float, _P, _P, _P, _P, c_int, _P, _LL, _P, _P],
+                                c_float, _P, _P, _P, _P, c_int, _P, _LL, _P, c_int, c_int, _P],
     "rllm_sink_attention_simt": [c_int, _P, _LL, _P, _P, _P, _LL, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int,
-                                 c_int, c_float, c_int, c_int, _P, _P, c_int, c_int, c_int, _P],
+                                 c_int, c_float, c_int, c_int, _P, _P, c_int, c_int, c_int, c_float, _P],
     "rllm_sink_attention_mma_supported": [c_int, c_int, c_int, c_int],
     "rllm_sink_attention_mma": [_P, _LL, _P, _P, _P, _LL, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-                                c_int, c_int, c_float, c_int, c_int, _P, _P, c_int, c_int, _P, _P, c_int, c_int, _P],
-    "rllm_postnorm": [_P, _P, c_int, _P, _P, c_int, c_float, _P, c_int, c_int, c_float, _P, c_int, _P],
+                                c_int, c_int, c_float, c_int, c_int, _P, _P, c_int, c_int, _P, _P, c_int, c_int, c_float, _P],
+    "rllm_postnorm": [_P, _P, c_int, _P, _P, c_int, c_float, _P, c_int, c_int, c_float, _P, c_int, c_int, _P],
     "rllm_cast_rows": [_P, _P, _LL, _P],
     "rllm_gated_act": [_P, c_int, _LL, _P, c_int, c_int, c_int, c_int, _P, _P],
     "rllm_relu2": [_P, c_int, _LL, _P],
@@ -55,10 +55,13 @@ def _caches(kcache, vcache, dtype, nkv=None):
 def qk_norm_rope_store(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, nh: int, nkv: int, kd: int, vd: int,
                        rot: int, wq: torch.Tensor | None, wk: torch.Tensor | None, eps: float,
                        table: torch.Tensor | None, slots: torch.Tensor | None, kcache: torch.Tensor | None,
-                       vcache: torch.Tensor | None, vfirst: torch.Tensor | None = None, lam: torch.Tensor | None = None) -> None:
+                       vcache: torch.Tensor | None, vfirst: torch.Tensor | None = None, lam: torch.Tensor | None = None,
+                       row_norm: bool = False, interleaved: bool = False) -> None:
     """proj [T, cols] holds q (nh heads of kd at q_off), k (nkv of kd at k_off) and v (nkv of vd at v_off). Per
     head: q and k divided by their root mean square times `wq` / `wk` (float [kd]; None: no norm), then the
-    first `rot` dimensions rotated (dimension i with i + rot/2) by `table` float [T, rot/2, 2] (cos, sin); q is
+    first `rot` dimensions rotated (dimension i with i + rot/2, or `interleaved` 2i with 2i + 1) by `table` float
+    [T, rot/2, 2] (cos, sin). `row_norm`: the root mean square is that of a token's whole query (key) row, all heads
+    together, and `wq` / `wk` hold a weight per number of it (float [nh * kd] / [nkv * kd]). q is
     written back in place, k and v go to their pages at `slots` (None, or -1 for a token: not stored). `vfirst` (rows of
     proj's type, [T, nkv * vd], a view with a longer row stride is fine) and `lam` (one float32 on the device): what is
     stored as the value is (1 - lam) v + lam vfirst, formed in float and rounded once; proj keeps v as it was."""
@@ -67,9 +70,9 @@ def qk_norm_rope_store(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, n
     need = max(q_off + nh * kd, k_off + nkv * kd, v_off + nkv * vd)
     if proj.dim() != 2 or proj.stride(1) != 1 or proj.shape[1] < need:
         raise KernelError(f"proj must be [T, >= {need}] with unit inner stride, got {list(proj.shape)}")
-    for w, n in ((wq, "query norm weight"), (wk, "key norm weight")):
+    for w, n, heads in ((wq, "query norm weight", nh), (wk, "key norm weight", nkv)):
         if w is not None:
-            _f32(w, n, (kd,))
+            _f32(w, n, (heads * kd if row_norm else kd,))
     if rot:
         if table is None:
             raise KernelError("a rotation needs the step's table of cos and sin")
@@ -93,7 +96,7 @@ def qk_norm_rope_store(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, n
         _dt(proj, "proj"), proj.data_ptr(), proj.stride(0), q_off, k_off, v_off, T, nh, nkv, kd, vd, rot, _ptr(wq),
         _ptr(wk), float(eps), _ptr(table) if rot else None, _ptr(slots), _ptr(kcache) if slots is not None else None,
         _ptr(vcache) if slots is not None else None, page_size, _ptr(vfirst), 0 if vfirst is None else vfirst.stride(0),
-        _ptr(lam), _stream()), "qk_norm_rope_store")
+        _ptr(lam), int(bool(row_norm)), int(bool(interleaved)), _stream()), "qk_norm_rope_store")
 
 
 def _attention_args(q, kcache, vcache, token_seq, positions, block_table, nh, sinks, gate):
@@ -120,20 +123,23 @@ def _attention_args(q, kcache, vcache, token_seq, positions, block_table, nh, si
 
 
 def sink_attention_simt(q, kcache, vcache, token_seq, positions, block_table, nh, scale, window=None, chunk=None,
-                        sinks=None, gate=None, keep_first: int = 0, sigmoid: bool = False) -> torch.Tensor:
+                        sinks=None, gate=None, keep_first: int = 0, sigmoid: bool = False,
+                        softcap: float | None = None) -> torch.Tensor:
     """Attention of every query row over its sequence's pages, in float on the CUDA cores. q [T, nh * kd] (a view
     with a longer row stride is fine); kcache [pages, nkv, page, kd]; vcache [pages, nkv, page, vd] -> [T, nh * vd]
     of q's dtype. A query at position p sees j <= p with j > p - window (if `window`) and j // chunk == p // chunk
     (if `chunk`), and besides every j <= p below `keep_first`. `sinks` float [nh]: exp(sink) joins the denominator.
     `sigmoid`: no softmax, a visible key's weight is sigmoid(score + sinks[head]) (`sinks` None: no bias). `gate` float
-    [T, >= nh]: logits of the output gate."""
+    [T, >= nh]: logits of the output gate. `softcap`: scores are bounded, softcap * tanh(score / softcap), before the mask
+    and the weights (a sink or a bias is not)."""
     T, nkv, page_size, kd, vd = _attention_args(q, kcache, vcache, token_seq, positions, block_table, nh, sinks, gate)
     out = torch.empty((T, nh * vd), dtype=q.dtype, device=q.device)
     _check(_fn("sink", "rllm_sink_attention_simt")(
         _dt(q, "q"), q.data_ptr(), q.stride(0), kcache.data_ptr(), vcache.data_ptr(), out.data_ptr(), out.stride(0),
         token_seq.data_ptr(), positions.data_ptr(), block_table.data_ptr(), block_table.stride(0), T, nh, nkv, kd, vd,
         page_size, float(scale), int(window or 0), int(chunk or 0), _ptr(sinks), _ptr(gate),
-        0 if gate is None else gate.stride(0), int(keep_first or 0), int(bool(sigmoid)), _stream()), "sink_attention_simt")
+        0 if gate is None else gate.stride(0), int(keep_first or 0), int(bool(sigmoid)), float(softcap or 0.0), _stream()),
+        "sink_attention_simt")
     return out
 
 
@@ -144,12 +150,12 @@ def mma_supported(dtype: torch.dtype, kd: int, vd: int, page_size: int) -> bool:
 
 def sink_attention_mma(q, kcache, vcache, token_seq, positions, block_table, cu_q, num_seqs, max_q_len, nh, scale,
                        window=None, chunk=None, sinks=None, gate=None, splits: int = 1, max_keys: int = 0,
-                       keep_first: int = 0, sigmoid: bool = False) -> torch.Tensor:
+                       keep_first: int = 0, sigmoid: bool = False, softcap: float | None = None) -> torch.Tensor:
     """The same attention in bfloat16 on the tensor cores (`mma.sync`, float softmax): row tiles of 64 (query,
     head-of-a-group) rows per sequence and kv head; `splits` > 1 deals a tile's keys out to that many CTAs in
     fixed ranges (steps of few rows) whose parts a second kernel merges in order. `cu_q` int32 [num_seqs + 1];
-    `max_keys`: a bound of the keys any query of the step sees (what `splits` cuts up). `keep_first`, `sigmoid`: as in
-    `sink_attention_simt`."""
+    `max_keys`: a bound of the keys any query of the step sees (what `splits` cuts up). `keep_first`, `sigmoid`,
+    `softcap`: as in `sink_attention_simt`."""
     T, nkv, page_size, kd, vd = _attention_args(q, kcache, vcache, token_seq, positions, block_table, nh, sinks, gate)
     if not mma_supported(q.dtype, kd, vd, page_size):
         raise KernelError(f"sink_attention_mma: bfloat16 with head sizes in steps of 16 up to 128, got {q.dtype} {kd}/{vd}")
@@ -165,7 +171,7 @@ def sink_attention_mma(q, kcache, vcache, token_seq, positions, block_table, cu_
         positions.data_ptr(), cu_q.data_ptr(), block_table.data_ptr(), block_table.stride(0), int(num_seqs), T,
         int(max_q_len), nh, nkv, kd, vd, page_size, float(scale), int(window or 0), int(chunk or 0), _ptr(sinks),
         _ptr(gate), 0 if gate is None else gate.stride(0), splits, _ptr(pacc), _ptr(pml), int(keep_first or 0),
-        int(bool(sigmoid)), _stream()), "sink_attention_mma", 2 if splits > 1 else 1)
+        int(bool(sigmoid)), float(softcap or 0.0), _stream()), "sink_attention_mma", 2 if splits > 1 else 1)
     return out
 
 
@@ -173,10 +179,11 @@ def sink_attention_mma(q, kcache, vcache, token_seq, positions, block_table, cu_
 
 def postnorm(h: torch.Tensor, y: torch.Tensor | None, alpha: float, w: torch.Tensor, eps: float,
              y2: torch.Tensor | None = None, y2_gate: torch.Tensor | None = None,
-             copy: torch.Tensor | None = None) -> torch.Tensor:
+             copy: torch.Tensor | None = None, output: bool = False) -> torch.Tensor:
     """h [T, H] float, in place: s = alpha * h + sum over parts of y ([T, H] or [T, parts, H] float, parts added in
     order) + sigmoid(y2_gate[t]) * y2[t] (y2 [T, H] float; y2_gate float [T, >= 1], its first column); then
-    h = w * s / sqrt(mean(s^2) + eps). `copy` [T, H] (bfloat16 or float32) also receives the new h."""
+    h = w * s / sqrt(mean(s^2) + eps). `copy` [T, H] (bfloat16 or float32) also receives the new h.
+    `output`: the norm is on the sublayer's output alone, s = the summands without h, and h += alpha * w * s / rms(s)."""
     _f32(h, "h")
     T, H = h.shape
     parts = 0
@@ -196,8 +203,8 @@ def postnorm(h: torch.Tensor, y: torch.Tensor | None, alpha: float, w: torch.Ten
             raise KernelError(f"postnorm: copy must be contiguous [{T}, {H}]")
     _check(_fn("sink", "rllm_postnorm")(h.data_ptr(), _ptr(y), parts, _ptr(y2), _ptr(y2_gate),
                                         0 if y2_gate is None else y2_gate.stride(0), float(alpha), w.data_ptr(), T, H,
-                                        float(eps), _ptr(copy), 0 if copy is None else _dt(copy, "copy"), _stream()),
-           "postnorm")
+                                        float(eps), _ptr(copy), 0 if copy is None else _dt(copy, "copy"), int(bool(output)),
+                                        _stream()), "postnorm")
     return h
 
 

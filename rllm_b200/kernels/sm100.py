@@ -29,9 +29,9 @@ ops.register_signatures("sm100", {
     "rllm_attention_fa": [_P, c_int, _P, _P, _P, c_int, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int,
                           c_int, c_int, c_float, c_int, c_int, _P, _P, _P],
     "rllm_attention_prefill_tc": [_P, c_int, _P, _P, _P, c_int, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int,
-                                  c_int, c_int, c_float, c_int, c_int, _P, _P, c_int, c_int, c_int, _P, c_int, _P],
+                                  c_int, c_int, c_float, c_int, c_int, _P, _P, c_int, c_int, c_int, c_float, _P, c_int, _P],
     "rllm_attention_decode": [_P, c_int, _P, _P, c_longlong, _P, c_int, _P, _P, c_int, c_int, c_int, c_int, c_int,
-                              c_int, c_float, c_int, c_int, _P, _P, c_int, c_int, _P, _P],
+                              c_int, c_float, c_int, c_int, _P, _P, c_int, c_float, c_int, _P, _P],
 })
 
 
@@ -126,7 +126,8 @@ def plan(epilogue: int, T: int, N: int, K: int, device="cuda:0", split: bool | i
 
 ACT_RELU2 = 1 << 8          # added to the store epilogue's number: max(value, 0)^2 is stored
 ACT_GELU_TANH = 2 << 8      # likewise: gelu(value) in its tanh form
-STORE_ACTS = {None: 0, "relu2": ACT_RELU2, "gelu_tanh": ACT_GELU_TANH}
+ACT_GELU_ERF = 3 << 8       # gelu(value) in its erf form
+STORE_ACTS = {None: 0, "relu2": ACT_RELU2, "gelu_tanh": ACT_GELU_TANH, "gelu_erf": ACT_GELU_ERF}
 
 
 def gemm(x: torch.Tensor, w: torch.Tensor, epilogue: int, out: torch.Tensor | None = None,
@@ -134,10 +135,10 @@ def gemm(x: torch.Tensor, w: torch.Tensor, epilogue: int, out: torch.Tensor | No
     """C = X W^T on the tensor cores. x [T, K] bf16 (unit inner stride); w [N, K] bf16 ([2N, K] with
     the SwiGLU epilogue). `out` is required for the accumulate epilogue (the float residual). `act`
     (store epilogue only; `relu2` True is act "relu2"): the activation of the float result is what is rounded and
-    stored: "relu2" max(., 0)^2, "gelu_tanh" gelu in its tanh form."""
+    stored: "relu2" max(., 0)^2, "gelu_tanh" gelu in its tanh form, "gelu_erf" in its erf form."""
     act = "relu2" if relu2 else act
     if act is not None and (epilogue != ops.EPI_STORE or act not in STORE_ACTS):
-        raise ops.KernelError("tc gemm: an activation (relu2, gelu_tanh) goes with the store epilogue only")
+        raise ops.KernelError("tc gemm: an activation (relu2, gelu_tanh, gelu_erf) goes with the store epilogue only")
     code = epilogue | STORE_ACTS[act]
     if not gemm_supported(x, w):
         raise ops.KernelError("tc gemm: operands must be bfloat16, K a multiple of 8, 16-byte aligned")
@@ -190,7 +191,7 @@ def gemm_norm(h: torch.Tensor, g: torch.Tensor, eps: float, w: torch.Tensor, epi
               rows: torch.Tensor | None = None, split: bool = True, act: str | None = None) -> torch.Tensor:
     """C = rmsnorm(h[rows]; g, eps) W^T in one kernel (store, store-float or SwiGLU epilogue; `act` as in `gemm`)."""
     if act is not None and (epilogue != ops.EPI_STORE or act not in STORE_ACTS):
-        raise ops.KernelError("tc gemm with norm: an activation (relu2, gelu_tanh) goes with the store epilogue only")
+        raise ops.KernelError("tc gemm with norm: an activation (relu2, gelu_tanh, gelu_erf) goes with the store epilogue only")
     if not norm_supported(h, g, w, rows):
         raise ops.KernelError("tc gemm with norm: float32 rows of K % 8 == 0 values, at most "
                               f"{norm_max_tokens()} tokens, bfloat16 weights, 16-byte aligned")
@@ -348,12 +349,13 @@ def _extras(chunk, sinks, gate, nh, rows):
 
 
 def attention_prefill_tc(q, kcache, vcache, cu_q, kv_lens, block_table, max_q_len, nh, scale, window, out=None,
-                         chunk=None, sinks=None, gate=None, keep_first=0, sigmoid=False):
+                         chunk=None, sinks=None, gate=None, keep_first=0, sigmoid=False, softcap=None):
     """Prefill attention on the tcgen05 tensor cores (bf16, head size 64 or 128): tiles of 128 rows x
     128 (64) keys, both products with their accumulators in TMEM. `chunk`: a query sees only the keys of its
     own block of that many positions; `sinks` float [nh]: exp(sink) joins a row's denominator; `gate` float
     logits [T, >= nh]: head h's output times sigmoid(gate[t, h]); `keep_first`: positions below it are seen whatever
-    the window says; `sigmoid`: no softmax, a visible key's weight is sigmoid(score + sinks[head])."""
+    the window says; `sigmoid`: no softmax, a visible key's weight is sigmoid(score + sinks[head]); `softcap`: scores
+    bounded, softcap * tanh(score / softcap)."""
     if not prefill_tc_supported(q, kcache):
         raise ops.KernelError("attention_prefill_tc: bfloat16, head size 64 or 128, rows 16-byte aligned")
     st = init(q.device)
@@ -364,7 +366,7 @@ def attention_prefill_tc(q, kcache, vcache, cu_q, kv_lens, block_table, max_q_le
         q.data_ptr(), q.stride(0), kcache.data_ptr(), vcache.data_ptr(), out.data_ptr(), out.stride(0),
         cu_q.data_ptr(), kv_lens.data_ptr(), block_table.data_ptr(), block_table.stride(0), kv_lens.numel(),
         max_q_len, kcache.shape[0], nh, nkv, hd, page_size, float(scale), int(window or 0),
-        *_extras(chunk, sinks, gate, nh, q.shape[0]), int(keep_first or 0), int(bool(sigmoid)), st.err.data_ptr(),
+        *_extras(chunk, sinks, gate, nh, q.shape[0]), int(keep_first or 0), int(bool(sigmoid)), float(softcap or 0.0), st.err.data_ptr(),
         st.sm_count, ops._stream())
     ops._check(rc, "attention_prefill_tc")
     return out
@@ -401,9 +403,10 @@ def decode_splits(num_seqs: int, nkv: int, max_kv_len: int, sm_count: int) -> in
 
 
 def attention_decode(q, kcache, vcache, kv_lens, block_table, nh, scale, window, max_kv_len, splits=None,
-                     out=None, chunk=None, sinks=None, gate=None):
+                     out=None, chunk=None, sinks=None, gate=None, softcap=None):
     """Attention for a step in which every sequence brings one token: the ranges of a sequence's
-    keys are merged inside a thread-block cluster (bf16, head size 64 or 128, any page size)."""
+    keys are merged inside a thread-block cluster (bf16, head size 64 or 128, any page size). `softcap`: scores bounded,
+    softcap * tanh(score / softcap)."""
     st = init(q.device)
     num_pages, nkv, page_size, hd = kcache.shape
     S = kv_lens.numel()
@@ -420,7 +423,7 @@ def attention_decode(q, kcache, vcache, kv_lens, block_table, nh, scale, window,
     rc = ops._fn("sm100", "rllm_attention_decode")(
         q.data_ptr(), q.stride(0), kcache.data_ptr(), vcache.data_ptr(), num_pages, out.data_ptr(),
         out.stride(0), kv_lens.data_ptr(), block_table.data_ptr(), block_table.stride(0), S, nh, nkv, hd,
-        page_size, float(scale), int(window or 0), *_extras(chunk, sinks, gate, nh, S), int(splits), st.err.data_ptr(),
+        page_size, float(scale), int(window or 0), *_extras(chunk, sinks, gate, nh, S), float(softcap or 0.0), int(splits), st.err.data_ptr(),
         ops._stream())
     ops._check(rc, "attention_decode")
     return out

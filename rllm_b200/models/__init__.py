@@ -4,5 +4,6 @@ from . import zukotar  # registers Zukotar
 from . import livovik  # registers Livovik
 from . import bazulorn  # registers Bazulorn
 from . import purozen  # registers Purozen
+from . import danonex  # registers Danonex
 
-__all__ = ["LayerCall", "Model", "llama", "zukotar", "livovik", "bazulorn", "purozen"]
+__all__ = ["LayerCall", "Model", "llama", "zukotar", "livovik", "bazulorn", "purozen", "danonex"]

@@ -5,7 +5,7 @@ from .norm import RMSNorm
 from .rope import InterleavedRotary, RotaryEmbedding, inverse_frequencies
 from .attention import GQAttention, SinkGQAttention, TalkingHeadsAttention
 from .ffn import ActFFN, GluFFN, SwiGLU
-from .block import GatedPreNormBlock, LoopStep, ParallelBlock, PostNormBlock, PreNormBlock, SandwichBlock
+from .block import GatedPreNormBlock, LoopStep, OutputNormBlock, ParallelBlock, PostNormBlock, PreNormBlock, SandwichBlock
 from .latent_attention import LatentAttention, LatentCacheSpec
 from .gla import GatedLinearAttention
 from .moe import GatedRoutedExperts, GluRoutedExperts, RoutedExperts
@@ -20,4 +20,4 @@ __all__ = ["CacheKind", "cache_kind_of", "register_cache_kind", "register_rope_r
            "LatentCacheSpec", "GatedLinearAttention", "RoutedExperts", "Summands", "SinkGQAttention", "ActFFN",
            "PostNormBlock", "GatedRoutedExperts", "NormedSum", "TalkingHeadsAttention", "GluFFN", "ParallelBlock",
            "GluRoutedExperts", "DeltaRuleMixer", "SideBySideMixer", "StateSpaceMixer", "PairEmbedding", "ScaledSum",
-           "GatedPreNormBlock", "MinGRUMixer"]
+           "GatedPreNormBlock", "MinGRUMixer", "OutputNormBlock"]

@@ -78,11 +78,15 @@ class SinkGQAttention(Part):
       numbers shared by all heads (tensors `q.norm`, `k.norm`), before the rotation;
       `qk_norm_weight` False: no weights, queries and keys become vectors of root mean square 1 (a plain factor
       commutes with the rotation, so it is the same norm whether a design names it before or after the rotation);
-    * `position`: a rotary part (its `rot_dim` leading dimensions of a head are rotated, the rest pass) or None;
+      `qk_norm_span` "row": the root mean square is that of a token's whole query (key) projection, all heads together,
+      and the weights have a number per row of the projection;
+    * `position`: a rotary part (its `rotated` leading dimensions of a head turn, in pairs half that width apart or
+      interleaved as the part says, the rest pass) or None;
     * the mask: causal, and a `window` (the last `window` positions) and/or a `chunk` (only the positions of the
       query's own block of `chunk` positions, blocks counted from position 0); `keep_first`: the positions below
       this number stay visible to every later query whatever the window says (their pages are never given back);
     * `sink`: one learned number per head (tensor `sink`) whose exponential joins the softmax's denominator;
+    * `softcap`: scores are bounded before mask and softmax, score <- softcap tanh(score / softcap); the sink is not;
     * `weights` "sigmoid": no softmax; a visible key's weight is sigmoid(score + b_h) with one learned number per
       head (tensor `score_bias`, None: no bias), not normalised over the keys;
     * `value_mix`: None, or (role, key). The values of the layers that share a `key` are mixed with those of the
@@ -99,7 +103,8 @@ class SinkGQAttention(Part):
                  position: Part | None = None, scale: float | None = None, window: int | None = None,
                  chunk: int | None = None, qk_norm: bool = False, sink: bool = False, gate: bool = False,
                  eps: float = 1e-6, names=("q", "k", "v", "o"), qk_norm_weight: bool = True, keep_first: int = 0,
-                 weights: str = "softmax", score_bias: str | None = None, value_mix: tuple | None = None):
+                 weights: str = "softmax", score_bias: str | None = None, value_mix: tuple | None = None,
+                 qk_norm_span: str = "head", softcap: float | None = None):
         if heads % kv_heads:
             raise ValueError(f"heads {heads} must be a multiple of kv_heads {kv_heads}")
         v_dim = head_dim if v_dim is None else v_dim
@@ -117,6 +122,11 @@ class SinkGQAttention(Part):
             raise ValueError(f"value_mix role {value_mix[0]!r} is not known (known: 'first', 'mix')")
         self.qk_norm_weight, self.keep_first, self.weights = qk_norm_weight, int(keep_first or 0), weights
         self.score_bias, self.value_mix = score_bias, value_mix
+        if qk_norm_span not in ("head", "row"):
+            raise ValueError(f"qk_norm_span {qk_norm_span!r} is not known (known: 'head', 'row')")
+        if softcap is not None and softcap <= 0:
+            raise ValueError(f"softcap must be above 0, got {softcap}")
+        self.qk_norm_span, self.softcap = qk_norm_span, None if softcap is None else float(softcap)
         self.w_qkv = self.w_o = self.w_g = self.q_norm = self.k_norm = self.sinks = self.bias = self.lam = None
 
     def children(self):
@@ -128,8 +138,9 @@ class SinkGQAttention(Part):
         ps = [Param("w_qkv", (Source(q, (H * D, W)), Source(k, (G * D, W)), Source(v, (G * V, W)))),
               Param("w_o", (Source(o, (W, H * V)),))]
         if self.qk_norm and self.qk_norm_weight:
-            ps += [Param("q_norm", (Source(q + ".norm", (D,), init="norm"),), role="vector"),
-                   Param("k_norm", (Source(k + ".norm", (D,), init="norm"),), role="vector")]
+            nq, nk = (D, D) if self.qk_norm_span == "head" else (H * D, G * D)
+            ps += [Param("q_norm", (Source(q + ".norm", (nq,), init="norm"),), role="vector"),
+                   Param("k_norm", (Source(k + ".norm", (nk,), init="norm"),), role="vector")]
         if self.sink:
             ps.append(Param("sinks", (Source("sink", (H,)),), role="vector"))
         if self.weights == "sigmoid" and self.score_bias is not None:
@@ -150,7 +161,9 @@ class SinkGQAttention(Part):
         f32 = lambda t: None if t is None else t.float().contiguous()
         self._qn, self._kn, self._sinks = f32(self.q_norm), f32(self.k_norm), f32(self.sinks)
         if self.qk_norm and not self.qk_norm_weight:
-            self._qn = self._kn = torch.ones(self.head_dim, dtype=torch.float32, device=device)
+            row = self.qk_norm_span == "row"
+            self._qn = torch.ones(self.head_dim * (self.heads if row else 1), dtype=torch.float32, device=device)
+            self._kn = torch.ones(self.head_dim * (self.kv_heads if row else 1), dtype=torch.float32, device=device)
         if self.weights == "sigmoid":
             self._sinks = f32(self.bias)
         self._lam = None if self.lam is None else self.lam.float().reshape(1).contiguous()
@@ -171,10 +184,11 @@ class SinkGQAttention(Part):
                 first, lam = ctx.per_forward.get(("value_mix", key)), self._lam
                 if first is None or first.shape[1] != G * V:
                     raise ValueError(f"{self.prefix}: the values to mix in ({key!r}) are missing or of another size")
-        be.qk_norm_rope_store(proj, 0, H * D, (H + G) * D, H, G, D, V, 0 if pos is None else pos.rot_dim,
-                              self._qn, self._kn, self.eps, None if pos is None else pos.table(ctx), cache, first, lam)
+        be.qk_norm_rope_store(proj, 0, H * D, (H + G) * D, H, G, D, V, 0 if pos is None else pos.rotated,
+                              self._qn, self._kn, self.eps, None if pos is None else pos.table(ctx), cache, first, lam,
+                              self.qk_norm_span == "row", pos is not None and pos.interleaved)
         att = be.sink_attention(proj[:, : H * D], cache, ctx, H, self.scale, self.window, self.chunk, self._sinks, gate,
-                                self.keep_first if self.window else 0, self.weights == "sigmoid")
+                                self.keep_first if self.window else 0, self.weights == "sigmoid", self.softcap)
         if residual is None:
             return be.linear_f32(att, self.w_o, tag="o")
         be.linear_residual(att, self.w_o, residual)

@@ -3,7 +3,8 @@ order (src/model/registry/llama.rs:163-245): h += mixer(norm(h)); h += ffn(norm(
 `SandwichBlock` norms each sublayer's output as well: h += norm_b(mixer(norm(h))), the same for
 the feed-forward, which may be absent. `LoopStep` is a block that only adds a learned vector to
 every row: what a pass of a looped stretch of layers begins with. `PostNormBlock` norms after the sum,
-h = norm(alpha h + sublayer(h)), the sublayers reading the stream itself. `ParallelBlock` has one norm whose
+h = norm(alpha h + sublayer(h)), the sublayers reading the stream itself; `OutputNormBlock` norms the sublayer's output
+alone, h += coef * norm(sublayer(h)), the sublayers again reading the stream itself. `ParallelBlock` has one norm whose
 output both sublayers read: h += mixer(n) + ffn(n), n = norm(h). `GatedPreNormBlock` is the pre-norm order with a
 gate on each sublayer's way into the stream: h += sigmoid(W_g n + b_g) * sublayer(n), n = norm(h), W_g a square matrix."""
 from __future__ import annotations
@@ -137,18 +138,37 @@ class PostNormBlock(Part):
     def cache_spec(self):
         return self.mixer.cache_spec()
 
+    @staticmethod
+    def _finish(be, h, y, alpha, norm):
+        return be.postnorm(h, y, alpha, norm.weight_f32(), norm.eps)
+
     def forward(self, h, ctx, cache):
         """h: float32 residual stream [T, hidden], updated in place."""
         be = ctx.backend
         kept = ctx.per_forward.get("stream_copy")
         x = kept[1] if kept is not None and kept[0] is h else be.stream_copy(h)
         y = self.mixer.forward(x, ctx, cache, None)
-        x = be.postnorm(h, y, self.alpha, self.mixer_norm.weight_f32(), self.mixer_norm.eps)
+        x = self._finish(be, h, y, self.alpha, self.mixer_norm)
         if self.ffn is not None:
             y = self.ffn.forward(x, ctx, None)
-            x = be.postnorm(h, y, self.alpha, self.ffn_norm.weight_f32(), self.ffn_norm.eps)
+            x = self._finish(be, h, y, self.alpha, self.ffn_norm)
         ctx.per_forward["stream_copy"] = (h, x)        # what the next block's mixer reads
         return h
+
+
+class OutputNormBlock(PostNormBlock):
+    """h += coef * norm1(mixer(h)); h += coef * norm2(ffn(h)) (the feed-forward may be absent). As in `PostNormBlock` the
+    sublayers read the stream itself in the run's storage type; norm, coefficient and sum are one float kernel, which
+    also writes the copy that the next sublayer's products read."""
+    graph_safe = True
+
+    def __init__(self, mixer: Part, mixer_norm: Part, ffn: Part | None = None, ffn_norm: Part | None = None,
+                 coef: float = 1.0, names=("mix.", "mlp.")):
+        super().__init__(mixer, mixer_norm, ffn, ffn_norm, alpha=coef, names=names)
+
+    @staticmethod
+    def _finish(be, h, y, coef, norm):
+        return be.output_norm(h, y, coef, norm.weight_f32(), norm.eps)
 
 
 class ParallelBlock(Part):
@@ -280,6 +300,7 @@ class LoopStep(Part):
 register_part("block", "prenorm", PreNormBlock)
 register_part("block", "sandwich", SandwichBlock)
 register_part("block", "postnorm", PostNormBlock)
+register_part("block", "output_norm", OutputNormBlock)
 register_part("block", "parallel", ParallelBlock)
 register_part("block", "prenorm_gated", GatedPreNormBlock)
 register_part("block", "loop_step", LoopStep)

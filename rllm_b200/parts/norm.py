@@ -1,6 +1,7 @@
 """RMSNorm as a part. Formula and rounding: src/gpu/cuda/shaders/rms_norm.cu:78-115 of the
 reference (sum of squares and scaling in float, weight used as stored). `offset`: the checkpoint stores
-the weight minus this number (weights "around zero": offset 1); the sum is formed once, in float."""
+the weight minus this number (weights "around zero": offset 1); the sum is formed once, in float. `scale`: a
+number that multiplies the normed row (a design's factor on the logits, say), folded into the weight once, in float."""
 from __future__ import annotations
 
 from .base import Param, Part, Source, register_part
@@ -9,14 +10,15 @@ from .base import Param, Part, Source, register_part
 class RMSNorm(Part):
     graph_safe = True
 
-    def __init__(self, size: int, eps: float, weight_name: str = "weight", offset: float = 0.0):
+    def __init__(self, size: int, eps: float, weight_name: str = "weight", offset: float = 0.0, scale: float = 1.0):
         self.size, self.eps, self.weight_name, self.offset = size, float(eps), weight_name, float(offset)
+        self.scale = float(scale)
         self.weight = self.stored = None
 
     def params(self):
-        if self.offset:
+        if self.offset or self.scale != 1.0:
             # what the checkpoint holds is bound to `stored`; `weight` is made from it when the weights are bound
-            return [Param("stored", (Source(self.weight_name, (self.size,), init="normal"),), role="vector")]
+            return [Param("stored", (Source(self.weight_name, (self.size,), init="normal" if self.offset else "norm"),), role="vector")]
         return [Param("weight", (Source(self.weight_name, (self.size,), init="norm"),), role="vector")]
 
     def forward(self, h, ctx):
@@ -36,8 +38,8 @@ class RMSNorm(Part):
 
     def finalize(self, device, dtype):
         self._w32 = None            # weights were (re)bound
-        if self.offset:
-            self.weight = (self.stored.float() + self.offset).contiguous()
+        if self.offset or self.scale != 1.0:
+            self.weight = ((self.stored.float() + self.offset) * self.scale).contiguous()
 
     def forward_f32(self, h, ctx):
         import torch

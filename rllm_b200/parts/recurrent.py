@@ -16,6 +16,8 @@ head and key channel g = exp(-exp(A_log) softplus(W_a2 (W_a1 h) + dt_bias)); per
     S <- diag(g) S;   u = beta (v - S^T k);   S <- S + k u^T;   o = S^T q.
 Each head's o is RMS-normed over vdim with one weight shared by the heads, times sigmoid(W_g2 (W_g1 h)), then W_o.
 The widths of the two bottlenecks are sizes of the checkpoint unless given (random-weights mode).
+`decay` "head": one decay per head, from a full projection, g = exp(-exp(A_log) softplus(W_a h + dt_bias)). `gate` "full":
+the output gate is silu(W_g h), from a full projection.
 
 `MinGRUMixer` (a gated recurrence whose gates read only the current token; no convolution, the state one number per
 channel). z = sigmoid(W_z h + b_z), u = W_x h + b_x, the candidate c = u + 1/2 where u >= 0 and sigmoid(u) where u < 0;
@@ -83,12 +85,16 @@ class DeltaRuleMixer(Part):
     returns_output = True
 
     def __init__(self, hidden: int, heads: int, kv_heads: int, dim: int, vdim: int, taps: int = 4, eps: float = 1e-6,
-                 unit_eps: float = 1e-6, decay_rank: int | None = None, gate_rank: int | None = None):
+                 unit_eps: float = 1e-6, decay_rank: int | None = None, gate_rank: int | None = None,
+                 decay: str = "channel", gate: str = "low_rank"):
         if heads % kv_heads:
             raise ValueError(f"heads {heads} must be a multiple of kv_heads {kv_heads}")
         self.hidden, self.heads, self.kv_heads, self.dim, self.vdim = hidden, heads, kv_heads, dim, vdim
         self.taps, self.eps, self.unit_eps = taps, float(eps), float(unit_eps)
         self.decay_rank, self.gate_rank = decay_rank, gate_rank
+        if decay not in ("channel", "head") or gate not in ("low_rank", "full"):
+            raise ValueError(f"delta rule: decay {decay!r} (known: 'channel', 'head') or gate {gate!r} (known: 'low_rank', 'full')")
+        self.decay, self.gate = decay, gate
         self.qk = kv_heads * dim
         self.conv_channels = 2 * self.qk + heads * vdim
         self.w_in = self.conv_w = self.w_b = self.a_log = self.w_norm = self.w_a2 = self.dt_bias = self.w_g2 = self.w_o = None
@@ -97,17 +103,23 @@ class DeltaRuleMixer(Part):
         W, H, QK, V = self.hidden, self.heads, self.qk, self.heads * self.vdim
         ra = -1 if self.decay_rank is None else self.decay_rank
         rg = -1 if self.gate_rank is None else self.gate_rank
-        return [Param("w_in", (Source("q", (QK, W)), Source("k", (QK, W)), Source("v", (V, W)), Source("a1", (ra, W)),
-                               Source("g1", (rg, W)))),
-                Param("conv_w", (Source("q.conv", (QK, self.taps)), Source("k.conv", (QK, self.taps)),
-                                 Source("v.conv", (V, self.taps))), role="vector"),
-                Param("w_b", (Source("b", (H, W)),)),
-                Param("a_log", (Source("A_log", (H,)),), role="vector"),
-                Param("w_norm", (Source("norm", (self.vdim,), init="norm"),), role="vector"),
-                Param("w_a2", (Source("a2", (H * self.dim, ra)),)),
-                Param("dt_bias", (Source("dt_bias", (H * self.dim,)),), role="vector"),
-                Param("w_g2", (Source("g2", (V, rg)),)),
-                Param("w_o", (Source("o", (W, V)),))]
+        channel, low = self.decay == "channel", self.gate == "low_rank"
+        first = [Source("q", (QK, W)), Source("k", (QK, W)), Source("v", (V, W))]
+        first += [Source("a1", (ra, W))] if channel else []
+        first += [Source("g1", (rg, W))] if low else [Source("g", (V, W))]
+        ps = [Param("w_in", tuple(first)),
+              Param("conv_w", (Source("q.conv", (QK, self.taps)), Source("k.conv", (QK, self.taps)),
+                               Source("v.conv", (V, self.taps))), role="vector"),
+              # step sizes, and with one decay per head the decays' logits behind them: a product of a few rows
+              Param("w_b", (Source("b", (H, W)),) if channel else (Source("b", (H, W)), Source("a", (H, W)))),
+              Param("a_log", (Source("A_log", (H,)),), role="vector"),
+              Param("w_norm", (Source("norm", (self.vdim,), init="norm"),), role="vector")]
+        if channel:
+            ps.append(Param("w_a2", (Source("a2", (H * self.dim, ra)),)))
+        ps.append(Param("dt_bias", (Source("dt_bias", (H * self.dim if channel else H,)),), role="vector"))
+        if low:
+            ps.append(Param("w_g2", (Source("g2", (V, rg)),)))
+        return ps + [Param("w_o", (Source("o", (W, V)),))]
 
     def cache_spec(self):
         return StateSpec((("S", (self.heads, self.dim, self.vdim), torch.float32),
@@ -116,7 +128,8 @@ class DeltaRuleMixer(Part):
     def finalize(self, device, dtype):
         f32 = lambda t: t.float().contiguous()
         self._conv_w, self._dt_bias, self._a_log, self._norm = f32(self.conv_w), f32(self.dt_bias), f32(self.a_log), f32(self.w_norm)
-        self._ra, self._rg = self.w_a2.shape[1], self.w_g2.shape[1]
+        self._ra = self.w_a2.shape[1] if self.decay == "channel" else 0
+        self._rg = self.w_g2.shape[1] if self.gate == "low_rank" else self.heads * self.vdim
         if self.w_in.shape[0] != self.conv_channels + self._ra + self._rg:
             raise ValueError(f"{self.prefix}a1 and g1 have {self.w_in.shape[0] - self.conv_channels} rows together, a2 and g2 "
                              f"take {self._ra} and {self._rg}")
@@ -125,17 +138,23 @@ class DeltaRuleMixer(Part):
         be = ctx.backend
         x = x.tensor() if hasattr(x, "tensor") else x
         H, G, d, v, C = self.heads, self.kv_heads, self.dim, self.vdim, self.conv_channels
-        proj = be.linear(x, self.w_in, tag="in")                                  # [T, q | k | v | a1 | g1]
-        beta = be.linear_f32(x, self.w_b, tag="beta")                             # float logits [T, H]
+        proj = be.linear(x, self.w_in, tag="in")                                  # [T, q | k | v | a1 (decays per channel) | g1 or g]
+        beta = be.linear_f32(x, self.w_b, tag="beta")                             # float logits [T, H (+ H: the decays')]
         qkv = be.short_conv(proj, 0, C, self._conv_w, None, ctx, cache.state["tail"])
         be.unit_heads(qkv, 0, G, d, d ** -0.5, self.unit_eps)
         be.unit_heads(qkv, self.qk, G, d, 1.0, self.unit_eps)
-        z = be.linear_f32(proj[:, C: C + self._ra], self.w_a2, tag="decay")       # [T, H * dim]
-        _, decay = be.softplus_decay(z, 0, H * d, self._dt_bias, self._a_log)
+        if self.decay == "channel":
+            z = be.linear_f32(proj[:, C: C + self._ra], self.w_a2, tag="decay")   # [T, H * dim]
+            _, decay = be.softplus_decay(z, 0, H * d, self._dt_bias, self._a_log)
+        else:
+            _, decay = be.softplus_decay(beta, H, H, self._dt_bias, self._a_log)  # [T, H]
         o = be.state_scan(qkv[:, : self.qk], G, qkv[:, self.qk: 2 * self.qk], G, qkv[:, 2 * self.qk:], decay, H, d, v, ctx,
-                          cache.state["S"], beta=beta)
-        gate = be.linear_f32(proj[:, C + self._ra:], self.w_g2, tag="gate")       # float logits [T, H * vdim]
-        g = be.gated_norm(o.view(-1, H * v), gate, 0, self._norm, self.eps, H, gate_first=False, act="sigmoid")
+                          cache.state["S"], beta=beta[:, :H])
+        if self.gate == "low_rank":
+            gate = be.linear_f32(proj[:, C + self._ra:], self.w_g2, tag="gate")   # float logits [T, H * vdim]
+            g = be.gated_norm(o.view(-1, H * v), gate, 0, self._norm, self.eps, H, gate_first=False, act="sigmoid")
+        else:
+            g = be.gated_norm(o.view(-1, H * v), proj, C + self._ra, self._norm, self.eps, H, gate_first=False, act="silu")
         if residual is None:
             return be.linear_f32(g, self.w_o, tag="o")
         be.linear_residual(g, self.w_o, residual)

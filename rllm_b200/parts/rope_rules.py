@@ -1,12 +1,14 @@
 """Rules that turn the plain rotary frequencies f_i = theta^(-2i/d) into a model's own, by name.
 
 A rule is a function `(inverse frequencies as float64 list, the rule's parameters as a dict) ->
-list` and, optionally, a check of the parameters that raises ValueError. The name is what a
+list` (the dict also holds the rotation's `base` and `dims`) and, optionally, a check of the parameters that
+raises ValueError and a factor on all cosines and sines. The name is what a
 config.json carries in `rope_scaling.rope_type`; the configuration reader accepts exactly the
 registered names and the rotary part applies the rule, so another rule (another family's long
 context scheme) is one `register_rope_rule` call, from anywhere.
 
-Built in: "linear" (every frequency divided by `factor`) and "llama3", the three bands of the
+Built in: "linear" (every frequency divided by `factor`), "yarn" (slow frequencies divided by `factor`, fast ones kept,
+a ramp over the index between, and a factor on cosines and sines that grows with ln `factor`) and "llama3", the three bands of the
 reference's "yarn" kernel (src/gpu/cuda/shaders/rope.cu:233-251) with beta_fast =
 high_freq_factor and beta_slow = low_freq_factor. The reference parses `rope_scaling` for Llama
 (src/model/config.rs:724-746) but never applies it; here it is applied.
@@ -16,12 +18,14 @@ from __future__ import annotations
 import math
 from typing import Callable
 
-_RULES: dict[str, tuple[Callable, Callable | None]] = {}
+_RULES: dict[str, tuple[Callable, Callable | None, Callable | None]] = {}
 
 
 def register_rope_rule(name: str, rule: Callable[[list[float], dict], list[float]],
-                       check: Callable[[dict], None] | None = None) -> None:
-    _RULES[name] = (rule, check)
+                       check: Callable[[dict], None] | None = None,
+                       magnitude: Callable[[dict], float] | None = None) -> None:
+    """`magnitude`: a function of the rule's parameters that gives the factor on every cosine and sine (None: 1)."""
+    _RULES[name] = (rule, check, magnitude)
 
 
 def registered_rope_rules() -> list[str]:
@@ -33,6 +37,12 @@ def rope_rule(name: str) -> Callable[[list[float], dict], list[float]]:
         return _RULES[name][0]
     except KeyError:
         raise KeyError(f"no rotary frequency rule named {name!r}; registered: {registered_rope_rules()}") from None
+
+
+def rope_magnitude(name: str, params: dict) -> float:
+    """The factor a rule puts on every cosine and sine."""
+    rule = _RULES.get(name)
+    return 1.0 if rule is None or rule[2] is None else float(rule[2](params))
 
 
 def check_rope_rule(name: str, params: dict) -> None:
@@ -90,5 +100,35 @@ def _check_llama3(p):
         raise ValueError(f"rope_scaling: high_freq_factor must exceed low_freq_factor (got low={low}, high={high})")
 
 
+def _yarn(freqs, p):
+    """Frequency i turns original * f_i / (2 pi) times over the original context. Up to the index where that is `fast`
+    turns frequencies stay, from the index where it is `slow` on they are divided by `factor`, linear in the index
+    between; both indices are rounded outwards and kept inside 0 .. dims - 1."""
+    dims, base, factor = int(p["dims"]), float(p["base"]), float(p["factor"])
+
+    def index(turns):
+        return dims * math.log(float(p["original"]) / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
+
+    lo = max(math.floor(index(float(p["fast"]))), 0)
+    hi = min(math.ceil(index(float(p["slow"]))), dims - 1)
+    out = []
+    for i, f in enumerate(freqs):
+        r = min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0)
+        out.append(f / factor * r + f * (1.0 - r))
+    return out
+
+
+def _check_yarn(p):
+    for key in ("factor", "original", "fast", "slow"):
+        v = p.get(key)
+        if isinstance(v, bool) or not isinstance(v, (int, float)) or v <= 0:
+            raise ValueError(f"yarn scaling of the rotation: {key!r} must be a number above 0, got {v!r}")
+
+
+def _yarn_magnitude(p):
+    return 0.1 * math.log(float(p["factor"])) + 1.0
+
+
 register_rope_rule("linear", _linear, _check_factor)
+register_rope_rule("yarn", _yarn, _check_yarn, _yarn_magnitude)
 register_rope_rule("llama3", _llama3, _check_llama3)
