@@ -213,17 +213,38 @@ def _purozen_sizes():
     return out
 
 
-BESIDE = {"bazulorn": "zukotar", "purozen": "bazulorn"}       # the design timed beside each one; Llama layers otherwise
+def _danonex_sizes():
+    """Four layers: attention, delta rule, delta rule, attention. Heads of 128 over four key/value heads, bounded scores
+    and a sink, half of each head rotated with scaled frequencies; as many delta-rule heads of 128 x 128 as the Bazulorn
+    layers beside it have, one query/key head for two of them; feed-forwards of four times the width everywhere. Beside
+    it four Bazulorn layers of equal width and heads in the same order (attention with mixed heads beside a state-space
+    recurrence, two delta-rule layers with a decay per channel, the first again) with dense gated feed-forwards of the
+    same weights (two thirds the inner size)."""
+    pz, out = _purozen_sizes(), {}
+    for name, W, H in (("w2048", 2048, 16), ("w4096", 4096, 32)):
+        ff = {"kind": "dense", "ff": 4 * W}
+        att = {"type": "attention", "mlp": ff, "mixer": {
+            "heads": H, "kv_heads": 4, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "softcap": 30.0,
+            "rot": {"base": 1000000.0, "dims": 64, "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}}
+        rec = {"type": "delta", "mlp": ff, "mixer": {"heads": H, "kv_heads": H // 2, "dim": 128, "vdim": 128, "conv": 4}}
+        out[name] = ({"architecture": "Danonex", "vocab": 32000, "width": W, "norm": {"eps": 1e-6}, "residual_mult": 0.5,
+                      "logit_scale": 2.0, "layers": [att, rec, rec, att]}, pz[name][1])
+    return out
+
+
+BESIDE = {"bazulorn": "zukotar", "purozen": "bazulorn", "danonex": "bazulorn"}       # the design timed beside each one; Llama layers otherwise
 
 
 def design_sizes(design):
     """name -> (the design's configuration, the layers beside it: Llama layers of equal width, depth and active
-    feed-forward weights, for Bazulorn the Zukotar model of equal width, depth, heads and experts, for Purozen
-    Bazulorn layers of equal width, depth and heads)."""
+    feed-forward weights, for Bazulorn the Zukotar model of equal width, depth, heads and experts, for Purozen and
+    Danonex Bazulorn layers of equal width, depth and heads)."""
     if design == "livovik":
         return _livovik_sizes()
     if design == "purozen":
         return _purozen_sizes()
+    if design == "danonex":
+        return _danonex_sizes()
     if design == "bazulorn":
         zk = design_sizes("zukotar")
         return {name: (cfg, zk[name][0]) for name, cfg in _bazulorn_sizes().items()}
@@ -325,9 +346,9 @@ def main():
     ap.add_argument("--workloads", default="", help="comma-separated: mixed_3b, continuous_8b, or all")
     ap.add_argument("--phase", default="all", choices=["all", "prefill", "decode"],
                     help="run one part only (for profiling; the JSON line then lacks the other parts)")
-    ap.add_argument("--designs", default="", choices=["", "zukotar", "livovik", "bazulorn", "purozen"],
+    ap.add_argument("--designs", default="", choices=["", "zukotar", "livovik", "bazulorn", "purozen", "danonex"],
                     help="instead of the default workload: prefill and decode of this design beside Llama layers of "
-                         "equal size (bazulorn: beside Zukotar layers; purozen: beside Bazulorn layers), random weights, "
+                         "equal size (bazulorn: beside Zukotar layers; purozen, danonex: beside Bazulorn layers), random weights, "
                          "with the time per operation; "
                          "prints its own JSON line")
     ap.add_argument("--profile-range", action="store_true",

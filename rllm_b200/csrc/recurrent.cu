@@ -24,7 +24,7 @@ using namespace rllm;
 
 namespace {
 
-constexpr int MAX_TAPS = 8;
+constexpr int MAX_TAPS = 16;
 
 __device__ __forceinline__ void cp_async4(float* smem, const float* gmem, bool pred) {      // pred false: zero
   const unsigned d = (unsigned)__cvta_generic_to_shared(smem);

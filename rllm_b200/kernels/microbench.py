@@ -11,6 +11,7 @@ ranges of keys) were tuned with, and the small case a profiler is pointed at.
     python -m rllm_b200.kernels.microbench latent-attn --heads 16 --rank 512 --rot 64 --batch 8 --context 1024
     python -m rllm_b200.kernels.microbench gla --heads 16 --dim 128 --vdim 128 --tokens 2048 [--batch 8]
     python -m rllm_b200.kernels.microbench sink --heads 32 --kv-heads 8 --dim 64 --vdim 48 --tokens 2048 --batch 8,64 --context 1024
+    python -m rllm_b200.kernels.microbench bounded --heads 16 --kv-heads 4 --dim 128 --vdim 128 --tokens 2048 --batch 8,64
     ... --plain 3      # no timing: three plain launches and a synchronize (for ncu -k ... -c ...)
 
 Timing: the kernel runs back to back over `--copies` distinct weight (or cache) tensors, larger
@@ -492,6 +493,88 @@ def cmd_gated(a) -> None:
     sm100.check_error(DEV)
 
 
+def cmd_bounded(a) -> None:
+    """The kernels of layers that norm a sublayer's output and attend with bounded scores, each beside its like kernel at
+    the same sizes: attention with a bound and a sink beside the same kernel without the bound, query/key norm over a
+    whole row with interleaved pairs beside the norm per head with pairs half a head apart, the norm of a sublayer's
+    output beside the norm of the sum, the erf gelu in a product's epilogue beside the tanh form and relu squared there,
+    the delta rule with a decay per head beside a decay per channel."""
+    from . import hybrid, sink
+    nh, nkv, kd, vd, page, W, cap = a.heads, a.kv_heads, a.dim, a.vdim, a.page, a.width, a.softcap
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=DEV)
+    bf = lambda *shape: torch.randn(*shape, device=DEV, dtype=torch.bfloat16)
+    sinks, scale = torch.randn(nh, device=DEV), kd ** -0.5
+    equal = kd == vd and kd in (64, 128)
+    for T in a.tokens:                                   # one prompt of T tokens
+        pages = (T + page - 1) // page
+        kc, vc = bf(pages, nkv, page, kd), bf(pages, nkv, page, vd)
+        bt, cu, lens = torch.arange(pages, device=DEV, dtype=torch.int32).view(1, pages), i32([0, T]), i32([T])
+        q, out = bf(T, nh * kd), torch.empty(T, nh * vd, device=DEV, dtype=torch.bfloat16)
+        pos, seq = torch.arange(T, device=DEV, dtype=torch.int32), torch.zeros(T, device=DEV, dtype=torch.int32)
+        flops = nh * (kd + vd) * T * (T + 1.0)
+        tc = lambda c: sm100.attention_prefill_tc(q, kc, vc, cu, lens, bt, T, nh, scale, None, out=out, sinks=sinks, softcap=c)
+        mma = lambda c: sink.sink_attention_mma(q, kc, vc, seq, pos, bt, cu, 1, T, nh, scale, None, None, sinks, None, 1, T, softcap=c)
+        if a.plain:
+            run([(lambda: tc(cap)) if equal and not a.mma else (lambda: mma(cap))], a.plain, f"bounded attention T={T} heads of {kd}/{vd}")
+            sm100.check_error(DEV)
+            return
+        for name, fn in ((("tcgen05", tc),) if equal else ()) + (("mma.sync", mma),):
+            run([lambda: fn(cap)] * 4, 0, f"bounded attention ({name}) T={T} heads={nh}/{nkv} of {kd}/{vd}", flops=flops)
+            if name == "tcgen05":                        # a bound below most scores: the exponential form everywhere
+                run([lambda: fn(0.25)] * 4, 0, f"  scores beyond the bound ({name}) T={T}", flops=flops)
+            run([lambda: fn(None)] * 4, 0, f"  like: no bound ({name}) T={T}", flops=flops)
+        proj = bf(T, (nh + nkv) * kd + nkv * vd)
+        rot = kd // 2
+        table, slots = torch.randn(T, rot // 2, 2, device=DEV), torch.arange(T, device=DEV, dtype=torch.int32)
+        nbytes = 2.0 * proj.numel() * 2
+        for row, inter, label in ((True, True, "query/key norm over the row, interleaved rotation, cache write"),
+                                  (False, False, "  like: norm per head, halves")):
+            wq, wk = (torch.ones(n * kd if row else kd, device=DEV) for n in (nh, nkv))
+            run([lambda: sink.qk_norm_rope_store(proj, 0, nh * kd, (nh + nkv) * kd, nh, nkv, kd, vd, rot, wq, wk, 1e-6, table, slots,
+                                                 kc, vc, row_norm=row, interleaved=inter)] * 4, 0, f"{label} T={T}", nbytes=nbytes)
+        h, y, w = torch.randn(T, W, device=DEV), torch.randn(T, W, device=DEV), torch.ones(W, device=DEV)
+        copy = bf(T, W)
+        for output, label in ((True, "norm of the output into the stream"), (False, "  like: norm of the sum")):
+            run([lambda: sink.postnorm(h, y, 0.5, w, 1e-6, copy=copy, output=output)] * 4, 0, f"{label} T={T} width={W}", nbytes=T * W * 14)
+        x, wu = bf(T, W), bf(4 * W, W)
+        for act in ("gelu_erf", "gelu_tanh", "relu2"):
+            run([lambda act=act: sm100.gemm(x, wu, ops.EPI_STORE, act=act)] * 4, 0,
+                f"{'' if act == 'gelu_erf' else '  like: '}up product with {act} in its epilogue T={T} {W} -> {4 * W}", flops=2.0 * T * W * 4 * W)
+        _delta_pair(hybrid, 1, T, W)
+    for B in a.batch:                                    # B single tokens at context C
+        C = a.context
+        pages = (C + page - 1) // page
+        copies = max(1, min(8, int(2e9 // (B * pages * nkv * page * (kd + vd) * 2))))
+        caches = [(bf(B * pages, nkv, page, kd), bf(B * pages, nkv, page, vd)) for _ in range(copies)]
+        bt = torch.randperm(B * pages, device=DEV).to(torch.int32).view(B, pages).contiguous()
+        pos, seq, cu = i32([C - 1] * B), torch.arange(B, device=DEV, dtype=torch.int32), torch.arange(B + 1, device=DEV, dtype=torch.int32)
+        q, lens = bf(B, nh * kd), i32([C] * B)
+        sp = max(1, min(16, 4 * sm100.init(DEV).sm_count // (B * nkv * ((nh // nkv + 63) // 64)), C // 128))
+        for c in (cap, None):
+            label = f"{'bounded attention' if c else '  like: no bound'} {B} x 1 token, {C} keys, heads of {kd}/{vd}"
+            if equal and nh // nkv <= 16:
+                run([(lambda k=k: sm100.attention_decode(q, k[0], k[1], lens, bt, nh, scale, None, C, sinks=sinks, softcap=c)) for k in caches], 0,
+                    label + " (clusters)", nbytes=B * C * nkv * (kd + vd) * 2)
+            run([(lambda k=k: sink.sink_attention_mma(q, k[0], k[1], seq, pos, bt, cu, B, 1, nh, scale, None, None, sinks, None, sp, C,
+                                                      softcap=c)) for k in caches], 0, label + " (mma.sync)", nbytes=B * C * nkv * (kd + vd) * 2)
+        _delta_pair(hybrid, B, 1, W)
+    sm100.check_error(DEV)
+
+
+def _delta_pair(hybrid, S, n, W) -> None:
+    """S sequences of n tokens, heads of 128 x 128 as wide together as the model."""
+    H, d, v, T = max(1, W // 128), 128, 128, S * n
+    q, k = (torch.nn.functional.normalize(torch.randn(T, H // 2 or 1, d, device=DEV), dim=-1).view(T, -1) for _ in range(2))
+    x, beta = torch.randn(T, H * v, device=DEV), torch.randn(T, H, device=DEV)
+    cu, slots = torch.arange(S + 1, device=DEV, dtype=torch.int32) * n, torch.arange(S, device=DEV, dtype=torch.int32)
+    states = [torch.zeros(S, H, d, v, device=DEV) for _ in range(4)]
+    for per_head in (True, False):
+        decay = torch.rand(T, H if per_head else H * d, device=DEV) * 0.1 + 0.9
+        run([lambda s=s: hybrid.state_scan(q, H // 2 or 1, k, H // 2 or 1, x, decay, H, d, v, cu, S, slots, s, beta) for s in states], 0,
+            f"{'delta rule, a decay per head' if per_head else '  like: a decay per channel'} {S} x {n} tokens, {H} heads of {d} x {v}",
+            nbytes=T * H * (d + 2 * v) * 4 + decay.numel() * 4 + 2 * S * H * d * v * 4, flops=7.0 * T * H * d * v)
+
+
 def main(argv=None) -> int:
     ints = lambda s: [int(x) for x in s.split(",")]
     ap = argparse.ArgumentParser(prog="python -m rllm_b200.kernels.microbench", description=__doc__.split("\n\n")[0])
@@ -540,6 +623,14 @@ def main(argv=None) -> int:
     p.add_argument("--batch", type=ints, default=[8, 64])
     for k, v in (("heads", 16), ("kv-heads", 4), ("dim", 128), ("vdim", 128), ("page", 16), ("context", 1024), ("window", 1024),
                  ("keep-first", 64), ("width", 2048), ("channels", 0)):
+        p.add_argument("--" + k, type=int, default=v)
+    p = sub.add_parser("bounded")
+    p.add_argument("--plain", type=int, default=0, help="N plain launches of the prompt attention kernel instead of timing")
+    p.add_argument("--mma", action="store_true", help="with --plain: the mma.sync kernel where both take the sizes")
+    p.add_argument("--tokens", type=ints, default=[2048])
+    p.add_argument("--batch", type=ints, default=[8, 64])
+    p.add_argument("--softcap", type=float, default=30.0)
+    for k, v in (("heads", 16), ("kv-heads", 4), ("dim", 128), ("vdim", 128), ("page", 16), ("context", 1024), ("width", 2048)):
         p.add_argument("--" + k, type=int, default=v)
     p = sub.add_parser("talk")
     p.add_argument("--plain", type=int, default=0, help="N plain launches of the prompt kernel instead of timing")
@@ -593,7 +684,7 @@ def main(argv=None) -> int:
         return 1
     {"gemm": cmd_gemm, "attn-decode": cmd_attn_decode, "attn-prefill": cmd_attn_prefill, "sample": cmd_sample,
      "experts": cmd_experts, "latent-attn": cmd_latent_attn, "gla": cmd_gla, "sink": cmd_sink, "talk": cmd_talk,
-     "scan": cmd_scan, "gated": cmd_gated}[a.cmd](a)
+     "scan": cmd_scan, "gated": cmd_gated, "bounded": cmd_bounded}[a.cmd](a)
     return 0
 
 
