@@ -146,7 +146,7 @@ def test_plain_mechanisms_against_closed_forms():
     q = k.roll(1, 0).clone()                     # token t asks for key t - 1 (token 0 for a key that comes later)
     o = P.delta_steps(q, k, v, one, one)
     assert torch.allclose(o[1:, 0], v[:-1, 0]) and float(o[0].abs().max()) == 0.0
-    # the read-out sees the current write; a second write to the same key replaces the first
+    # what a token writes it also reads; a second write to the same key replaces the first
     assert torch.allclose(P.delta_steps(k, k, v, one, one), v)
     k2 = k[[0, 0]]
     assert torch.allclose(P.delta_steps(k2, k2, v[:2], one[:2], one[:2]), v[:2])
