@@ -58,7 +58,6 @@ struct DecParams {
   const float* sinks;   // per head, or null: exp(sink) joins the denominator (no key, no value)
   const float* gate;    // float logits [S, gate_ld] or null: head h's output times sigmoid(gate[seq, h])
   int gate_ld;
-  SoftCap cap;          // cap.c > 0: scores are bounded, cap tanh(score / cap), before mask and softmax (the sink is not)
 };
 
 // The last step of a row: the sink joins the denominator, the sum is divided, the gate applied.
@@ -132,10 +131,11 @@ template <int HD> struct DCfg {
 
 // MAXC: the most ranges (CTAs of a cluster) this instantiation merges, 8 or 16: the merge holds that many
 // addresses and maxima a thread
-template <int HD, int MAXC>
+// CAP: scores are bounded, cap tanh(score / cap), before mask and softmax (the sink is not)
+template <int HD, int MAXC, bool CAP>
 // (head size 64: 168 registers a thread; six warps twice per SM leave 170)
 __global__ void __launch_bounds__(DCfg<HD>::THREADS)
-attn_decode_kernel(const DecParams p) {
+attn_decode_kernel(const DecParams p, const SoftCap cap) {
   typedef DCfg<HD> C;
   constexpr int NW = C::NW, D = C::D, THREADS = C::THREADS;
   constexpr int TILE = C::TILE;
@@ -237,7 +237,6 @@ attn_decode_kernel(const DecParams p) {
     for (int i = 0; i < DTILES; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
     float mA = -INFINITY, mB = -INFINITY, lA = 0.f, lB = 0.f;
     const int mat = lane >> 3, rr = lane & 7;
-    const float sl = p.cap.c > 0.f ? 1.f : p.scale_log2e;
 
     for (int i = warp; i < n_tiles; i += NW) {
       cp_async_wait<D - 1>();                       // this warp's oldest group, tile i, has landed
@@ -265,11 +264,11 @@ attn_decode_kernel(const DecParams p) {
           mma16816(sc[2 * np + 1], qf[kk], kf[kk][np][2], kf[kk][np][3]);
         }
       }
-      if (p.cap.c > 0.f) {                             // bounded scores leave the bound in the log2 domain (sl is 1 then)
+      if (CAP) {                             // bounded scores leave the bound in the log2 domain
 #pragma unroll
         for (int nt = 0; nt < TILE / 8; ++nt) {
-          sc[nt][0] = softcap_log2(sc[nt][0], p.cap); sc[nt][1] = softcap_log2(sc[nt][1], p.cap);
-          if (G > 8) { sc[nt][2] = softcap_log2(sc[nt][2], p.cap); sc[nt][3] = softcap_log2(sc[nt][3], p.cap); }
+          sc[nt][0] = softcap_log2(sc[nt][0], cap); sc[nt][1] = softcap_log2(sc[nt][1], cap);
+          if (G > 8) { sc[nt][2] = softcap_log2(sc[nt][2], cap); sc[nt][3] = softcap_log2(sc[nt][3], cap); }
         }
       }
       // ---- the V fragments are asked for now and used after the softmax arithmetic
@@ -302,7 +301,7 @@ attn_decode_kernel(const DecParams p) {
       mxB = fmaxf(mxB, __shfl_xor_sync(0xffffffffu, mxB, 1));
       mxB = fmaxf(mxB, __shfl_xor_sync(0xffffffffu, mxB, 2));
       // running maximum in the exp2 domain (the scale is positive, so it commutes with max)
-      const float mnA = fmaxf(mA, mxA * sl), mnB = fmaxf(mB, mxB * sl);
+      const float mnA = fmaxf(mA, CAP ? mxA : mxA * p.scale_log2e), mnB = fmaxf(mB, CAP ? mxB : mxB * p.scale_log2e);
       const float useA = (mnA == -INFINITY) ? 0.f : mnA, useB = (mnB == -INFINITY) ? 0.f : mnB;
       if (__any_sync(0xffffffffu, mnA != mA || mnB != mB)) {      // a new maximum somewhere: rescale
         const float corrA = fast_exp2(mA - useA), corrB = fast_exp2(mB - useB);     // exp2(-inf) = 0
@@ -315,6 +314,7 @@ attn_decode_kernel(const DecParams p) {
       for (int kb = 0; kb < TILE / 16; ++kb) {
         uint32_t a[4];
         {
+          const float sl = CAP ? 1.f : p.scale_log2e;
           const float p0 = fast_exp2(fmaf(sc[2 * kb][0], sl, -useA)), p1 = fast_exp2(fmaf(sc[2 * kb][1], sl, -useA));
           const float p2 = fast_exp2(fmaf(sc[2 * kb][2], sl, -useB)), p3 = fast_exp2(fmaf(sc[2 * kb][3], sl, -useB));
           const float p4 = fast_exp2(fmaf(sc[2 * kb + 1][0], sl, -useA)), p5 = fast_exp2(fmaf(sc[2 * kb + 1][1], sl, -useA));
@@ -412,18 +412,18 @@ attn_decode_kernel(const DecParams p) {
 }
 
 // ------------------------------------------------------------------------------------ host side
-template <int HD, int MAXC>
-int launch_dec_c(const DecParams& p, int num_seqs, cudaStream_t s) {
+template <int HD, int MAXC, bool CAP>
+int launch_dec_c(const DecParams& p, const SoftCap& cap, int num_seqs, cudaStream_t s) {
   typedef DCfg<HD> C;
   static bool configured[64] = {};
-  if (allow_dynamic_smem(attn_decode_kernel<HD, MAXC>, C::smem_bytes(16), configured)) return -5;
+  if (allow_dynamic_smem(attn_decode_kernel<HD, MAXC, CAP>, C::smem_bytes(16), configured)) return -5;
   if (MAXC > 8) {
     // more than 8 CTAs in a cluster need the kernel's own permission, per device
     static bool wide[64] = {};
     int dev = 0;
     if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= 64) { cudaGetLastError(); return -5; }
     if (!wide[dev]) {
-      if (cudaFuncSetAttribute(attn_decode_kernel<HD, MAXC>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1) != cudaSuccess) {
+      if (cudaFuncSetAttribute(attn_decode_kernel<HD, MAXC, CAP>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1) != cudaSuccess) {
         cudaGetLastError();
         return ERR_BAD_SIZE;
       }
@@ -432,12 +432,14 @@ int launch_dec_c(const DecParams& p, int num_seqs, cudaStream_t s) {
   }
   dim3 grid(p.nkv, num_seqs, p.splits);
   if (grid.y > 65535) return ERR_TOO_LARGE;
-  return launch_ex(attn_decode_kernel<HD, MAXC>, grid, dim3(C::THREADS), C::smem_bytes(p.nh / p.nkv), s, p.splits, p);
+  return launch_ex(attn_decode_kernel<HD, MAXC, CAP>, grid, dim3(C::THREADS), C::smem_bytes(p.nh / p.nkv), s, p.splits, p, cap);
 }
 
 template <int HD>
-int launch_dec(const DecParams& p, int num_seqs, cudaStream_t s) {
-  return p.splits <= 8 ? launch_dec_c<HD, 8>(p, num_seqs, s) : launch_dec_c<HD, 16>(p, num_seqs, s);
+int launch_dec(const DecParams& p, const SoftCap& cap, int num_seqs, cudaStream_t s) {
+  if (cap.c > 0.f)
+    return p.splits <= 8 ? launch_dec_c<HD, 8, true>(p, cap, num_seqs, s) : launch_dec_c<HD, 16, true>(p, cap, num_seqs, s);
+  return p.splits <= 8 ? launch_dec_c<HD, 8, false>(p, cap, num_seqs, s) : launch_dec_c<HD, 16, false>(p, cap, num_seqs, s);
 }
 
 }  // namespace
@@ -446,7 +448,7 @@ int launch_dec(const DecParams& p, int num_seqs, cudaStream_t s) {
 // kcache / vcache: [num_pages][nkv][page_size][hd] bf16. kv_lens [S]: keys visible to each
 // sequence's token (its own included). splits: ranges of keys per sequence (1..16, one cluster).
 // chunk > 0: only the keys of the token's own block of `chunk` positions; sinks float [nh] or null; gate float
-// logits [S, gate_ld] or null; softcap > 0: bounded scores (see DecParams).
+// logits [S, gate_ld] or null; softcap > 0: bounded scores.
 // `err` is not used (this kernel has no wait that can run out); it keeps the launchers alike.
 RLLM_API int rllm_attention_decode(const void* q, int q_stride, const void* kcache, const void* vcache,
                                    long long num_pages, void* out, int out_stride, const int* kv_lens,
@@ -465,9 +467,9 @@ RLLM_API int rllm_attention_decode(const void* q, int q_stride, const void* kcac
   p.kv_lens = kv_lens; p.block_table = block_table; p.bt_stride = bt_stride; p.nh = nh; p.nkv = nkv;
   p.page_size = page_size; p.window = window; p.splits = splits; p.scale_log2e = scale * 1.4426950408889634f;
   p.chunk = chunk; p.sinks = sinks; p.gate = gate; p.gate_ld = gate_ld;
-  p.cap = make_softcap(softcap, scale);
   p.page_shift = -1;
   for (int sft = 0; sft < 31; ++sft) if ((1 << sft) == page_size) p.page_shift = sft;
   cudaStream_t s = (cudaStream_t)stream;
-  return hd == 64 ? launch_dec<64>(p, num_seqs, s) : launch_dec<128>(p, num_seqs, s);
+  const SoftCap cap = make_softcap(softcap, scale);
+  return hd == 64 ? launch_dec<64>(p, cap, num_seqs, s) : launch_dec<128>(p, cap, num_seqs, s);
 }

@@ -164,7 +164,8 @@ __device__ __forceinline__ void softcap_poly2(uint32_t& x0, uint32_t& x1, float 
 }
 
 // TMA: the K and V tiles come by tensor copies over the caches seen as [pages * kv heads][page size][HD].
-template <int HD, bool TMA>
+// CAP: scores are bounded (p.cap).
+template <int HD, bool TMA, bool CAP>
 __global__ void __launch_bounds__(THREADS, 1)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constant__ CUtensorMap tmap_v,
                        const PfParams p) {
@@ -466,8 +467,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_
     const uint32_t pv_addr = lane_addr + C::O_COL + (uint32_t)g * HD;
     const uint32_t prow = p_s + (uint32_t)g * C::P_BYTES + (uint32_t)(r * 128);
     constexpr int NC = PN / 32;                           // the row's scores come 32 at a time
-    const bool bounded = p.cap.c > 0.f;
-    const float sl = bounded ? 1.f : p.scale_log2e;        // bounded scores leave the bound in the log2 domain
+    const float sl = CAP ? 1.f : p.scale_log2e;        // bounded scores leave the bound in the log2 domain
     // m: what the exponentials are taken against, up to 2^8 behind the true maximum. A sink opens the row's
     // running softmax as a key of score `sink` (not scaled) and value zero.
     const bool sig = p.sigmoid != 0;
@@ -497,7 +497,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_
       tc_fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive(&s_free[k % SB]);        // the accumulator may take the scores of step k + 3
-      if (bounded) {
+      if (CAP) {
         float far[NC];
 #pragma unroll
         for (int c = 0; c < NC; ++c) {
@@ -685,11 +685,16 @@ int cache_map(CUtensorMap* out, const void* ptr, long long planes, int page_size
   return 0;
 }
 
+template <int HD, bool TMA, bool CAP>
+int launch_pf_c(const CUtensorMap& mk, const CUtensorMap& mv, const PfParams& p, int ctas, cudaStream_t s) {
+  static bool configured[64] = {};
+  if (allow_dynamic_smem(attn_prefill_tc_kernel<HD, TMA, CAP>, Shape<HD>::SMEM_BYTES, configured)) return -5;
+  return launch_ex(attn_prefill_tc_kernel<HD, TMA, CAP>, dim3(ctas), dim3(THREADS), Shape<HD>::SMEM_BYTES, s, 1, mk, mv, p);
+}
+
 template <int HD, bool TMA>
 int launch_pf(const CUtensorMap& mk, const CUtensorMap& mv, const PfParams& p, int ctas, cudaStream_t s) {
-  static bool configured[64] = {};
-  if (allow_dynamic_smem(attn_prefill_tc_kernel<HD, TMA>, Shape<HD>::SMEM_BYTES, configured)) return -5;
-  return launch_ex(attn_prefill_tc_kernel<HD, TMA>, dim3(ctas), dim3(THREADS), Shape<HD>::SMEM_BYTES, s, 1, mk, mv, p);
+  return p.cap.c > 0.f ? launch_pf_c<HD, TMA, true>(mk, mv, p, ctas, s) : launch_pf_c<HD, TMA, false>(mk, mv, p, ctas, s);
 }
 
 }  // namespace

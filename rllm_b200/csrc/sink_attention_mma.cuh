@@ -84,7 +84,8 @@ __device__ __forceinline__ int first_key(int pos, int window, int chunk) {
 // FEW: the step's sequences bring at most 16 rows each (single tokens with up to 16 heads a kv head). The four warps
 // then all hold the tile's 16 rows and split each tile's 64 keys between them (16 keys a warp), each with a running
 // softmax of its own; the four are joined in warp order through shared memory at the end.
-template <int DP, bool FEW, bool SIG>
+// CAP: scores are bounded (p.cap).
+template <int DP, bool FEW, bool SIG, bool CAP>
 __global__ void __launch_bounds__(THREADS) sink_attention_mma_kernel(const Args p) {
   pdl_launch();
   pdl_wait();
@@ -207,7 +208,6 @@ __global__ void __launch_bounds__(THREADS) sink_attention_mma_kernel(const Args 
     m1 = v1 ? 0.f : -INFINITY;
   }
 
-  const float sl = p.cap.c > 0.f ? 1.f : p.scale_log2;
   // STAGES - 1 tiles are on their way while one is worked on (a commit per tile, empty past the end, so that
   // the count of groups in flight says which tile has landed)
 #pragma unroll
@@ -243,7 +243,7 @@ __global__ void __launch_bounds__(THREADS) sink_attention_mma_kernel(const Args 
       }
     }
     // a bounded score leaves the bound in the log2 domain, where it needs no further scale
-    if (p.cap.c > 0.f) {
+    if (CAP) {
 #pragma unroll
       for (int nt = 0; nt < NT; ++nt) {
         sc[nt][0] = softcap_log2(sc[nt][0], p.cap); sc[nt][1] = softcap_log2(sc[nt][1], p.cap);
@@ -261,8 +261,8 @@ __global__ void __launch_bounds__(THREADS) sink_attention_mma_kernel(const Args 
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
           const int j = key0 + nt * 8 + (lane & 3) * 2 + e;
-          const float a = (v0 && (j >= st0 || j < p.keep_first) && j <= pos0) ? sc[nt][e] * sl : -INFINITY;
-          const float c = (v1 && (j >= st1 || j < p.keep_first) && j <= pos1) ? sc[nt][2 + e] * sl : -INFINITY;
+          const float a = (v0 && (j >= st0 || j < p.keep_first) && j <= pos0) ? (CAP ? sc[nt][e] : sc[nt][e] * p.scale_log2) : -INFINITY;
+          const float c = (v1 && (j >= st1 || j < p.keep_first) && j <= pos1) ? (CAP ? sc[nt][2 + e] : sc[nt][2 + e] * p.scale_log2) : -INFINITY;
           sc[nt][e] = a; sc[nt][2 + e] = c;
           mx0 = fmaxf(mx0, a); mx1 = fmaxf(mx1, c);
         }
@@ -271,7 +271,7 @@ __global__ void __launch_bounds__(THREADS) sink_attention_mma_kernel(const Args 
 #pragma unroll
       for (int nt = 0; nt < NT; ++nt) {
 #pragma unroll
-        for (int e = 0; e < 4; ++e) sc[nt][e] *= sl;
+        for (int e = 0; e < 4; ++e) if (!CAP) sc[nt][e] *= p.scale_log2;
         mx0 = fmaxf(mx0, fmaxf(sc[nt][0], sc[nt][1])); mx1 = fmaxf(mx1, fmaxf(sc[nt][2], sc[nt][3]));
       }
     }
@@ -468,13 +468,17 @@ RLLM_API int rllm_sink_attention_mma(const void* q, long long q_stride, const vo
   const int smem = 2 * STAGES * KEYS * (dp + 8) * (int)sizeof(bf16);     // also holds the FEW join: 4 x 16 x (dp + 2) floats
   const bool few = (long long)max_q_len * Gq <= 16;             // every sequence's rows fit one warp's 16
   int rc;
-#define GO(D, F, G)                                                                                     \
+#define GO(D, F, G, C)                                                                                  \
   {                                                                                                     \
     static bool done[64] = {};                                                                          \
-    if ((rc = allow_dynamic_smem(sink_attention_mma_kernel<D, F, G>, smem, done))) return rc;           \
-    rc = launch_ex(sink_attention_mma_kernel<D, F, G>, grid, dim3(THREADS), (size_t)smem, s, 1, a);     \
+    if ((rc = allow_dynamic_smem(sink_attention_mma_kernel<D, F, G, C>, smem, done))) return rc;           \
+    rc = launch_ex(sink_attention_mma_kernel<D, F, G, C>, grid, dim3(THREADS), (size_t)smem, s, 1, a);     \
   }
-#define GO2(D, F) { if (sigmoid) GO(D, F, true) else GO(D, F, false) }
+#define GO2(D, F)                                                            \
+  {                                                                           \
+    if (softcap > 0.f) { if (sigmoid) GO(D, F, true, true) else GO(D, F, false, true) } \
+    else { if (sigmoid) GO(D, F, true, false) else GO(D, F, false, false) }   \
+  }
   if (dp == 64) { if (few) GO2(64, true) else GO2(64, false) }
   else { if (few) GO2(128, true) else GO2(128, false) }
 #undef GO2

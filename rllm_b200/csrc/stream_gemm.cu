@@ -317,7 +317,7 @@ stream_gemm_kernel(const Params p) {
           float v = s0;
           if (p.act == 1) v = fmaxf(s0, 0.f) * fmaxf(s0, 0.f);
           else if (p.act == 2) v = s0 / (1.f + expf(-1.5957691216057308f * (s0 + 0.044715f * s0 * s0 * s0)));   // = 0.5 s (1 + tanh(.))
-          else if (p.act == 3) v = 0.5f * s0 * (1.f + erff(s0 * 0.7071067811865476f));
+          else if (p.act == 3) v = gelu_erf_fast(s0);
           ((bf16*)p.C)[o] = __float2bfloat16_rn(v);
         }
         else if (EPI == EPI_STORE_F32) ((float*)p.C)[o] = s0;

@@ -165,8 +165,25 @@ __device__ __forceinline__ float store_act(const Params& p, float v) {
   if (p.act == 1) { v = fmaxf(v, 0.f); v *= v; }
   // 0.5 v (1 + tanh(u)) = v / (1 + exp(-2u)), u = sqrt(2/pi) (v + 0.044715 v^3)
   else if (p.act == 2) v = __fdividef(v, 1.f + __expf(-1.5957691216057308f * (v + 0.044715f * v * v * v)));
-  else if (p.act == 3) v = 0.5f * v * (1.f + erff(v * 0.7071067811865476f));
+  else if (p.act == 3) v = gelu_erf_fast(v);
   return v;
+}
+// The same for a thread's N values at once: the branch on the activation lies outside the loop.
+template <int N>
+__device__ __forceinline__ void store_act_all(const Params& p, uint32_t (&g)[N]) {
+  if (p.act == 1) {
+#pragma unroll
+    for (int i = 0; i < N; ++i) { const float v = fmaxf(__uint_as_float(g[i]), 0.f); g[i] = __float_as_uint(v * v); }
+  } else if (p.act == 2) {
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+      const float v = __uint_as_float(g[i]);
+      g[i] = __float_as_uint(__fdividef(v, 1.f + __expf(-1.5957691216057308f * (v + 0.044715f * v * v * v))));
+    }
+  } else if (p.act == 3) {
+#pragma unroll
+    for (int i = 0; i < N; ++i) g[i] = __float_as_uint(gelu_erf_fast(__uint_as_float(g[i])));
+  }
 }
 
 template <int EPI>
@@ -1021,9 +1038,10 @@ tc_gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmap_w, const __gr
                 if (c0 + jj < lim) cp[(size_t)jj * p.ldc] = r[jj] + __uint_as_float(g[jj]);
             } else if (EPI == EPI_STORE) {
               bf16* cp = (bf16*)p.C + (size_t)(t0 + c0) * p.ldc + n;
+              store_act_all(p, g);
 #pragma unroll
               for (int jj = 0; jj < CW; ++jj, cp += p.ldc)
-                if (c0 + jj < lim) *cp = __float2bfloat16_rn(store_act(p, __uint_as_float(g[jj])));
+                if (c0 + jj < lim) *cp = __float2bfloat16_rn(__uint_as_float(g[jj]));
             } else {
 #pragma unroll
               for (int jj = 0; jj < CW; ++jj) {
