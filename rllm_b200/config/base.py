@@ -114,6 +114,43 @@ def load_config(model_dir: str) -> tuple[Architecture, ModelConfig]:
     return config_from_dict(raw)
 
 
+def require_object(raw: dict, key: str, where: str, optional: bool = False) -> dict | None:
+    v = raw.get(key)
+    if v is None:
+        if optional:
+            return None
+        raise ConfigError(f"{where} lacks required key {key!r}")
+    if not isinstance(v, dict):
+        raise ConfigError(f"{where}: {key!r} must be an object, got {v!r}")
+    return v
+
+
+def read_loop(raw: dict, n_layers: int) -> tuple[int, int, int]:
+    """(start, stop, times) of the key `loop`: layers start .. stop-1 run `times` times in a row; absent: (0, 0, 1)."""
+    loop = require_object(raw, "loop", "config.json", optional=True)
+    if loop is None:
+        return 0, 0, 1
+    start, stop = require_int(loop, "start", minimum=0), require_int(loop, "stop", minimum=0)
+    if not start < stop <= n_layers:
+        raise ConfigError(f"loop: start {start} < stop {stop} <= {n_layers} layers does not hold")
+    return start, stop, require_int(loop, "times", minimum=1)
+
+
+def looped_runs(n_layers: int, start: int, stop: int, times: int) -> list[tuple[int, int | None]]:
+    """[(layer, pass number if the run begins a pass of the loop, else None)] in running order (stop 0: no loop)."""
+    if stop <= start:
+        return [(i, None) for i in range(n_layers)]
+    runs = [(i, None) for i in range(start)]
+    for t in range(times):
+        runs += [(i, t if i == start else None) for i in range(start, stop)]
+    return runs + [(i, None) for i in range(stop, n_layers)]
+
+
+def read_eos(raw: dict) -> tuple[int, ...]:
+    eos = raw.get("eos_token_id")
+    return () if eos is None else tuple(int(e) for e in (eos if isinstance(eos, (list, tuple)) else (eos,)))
+
+
 def require_int(raw: dict, key: str, *, minimum: int = 1, default: int | None = None) -> int:
     v = raw.get(key, default)
     if v is None:

@@ -21,18 +21,8 @@ from __future__ import annotations
 from dataclasses import dataclass
 from typing import Any
 
-from .base import ConfigError, ModelConfig, require_float, require_int
-
-
-def _obj(raw: dict, key: str, where: str, optional: bool = False):
-    v = raw.get(key)
-    if v is None:
-        if optional:
-            return None
-        raise ConfigError(f"{where} lacks required key {key!r}")
-    if not isinstance(v, dict):
-        raise ConfigError(f"{where}: {key!r} must be an object, got {v!r}")
-    return v
+from .base import ConfigError, ModelConfig, looped_runs, read_loop, require_float, require_int
+from .base import require_object as _obj
 
 
 @dataclass(frozen=True)
@@ -159,14 +149,7 @@ class ZukotarConfig(ModelConfig):
             if mlp is not None and not isinstance(mlp, dict):
                 raise ConfigError(f"{where}: 'mlp' must be an object or null")
             layers.append(ZukotarLayer(L["type"], mixer, None if mlp is None else MoEConfig.from_dict(mlp, where + ".mlp")))
-        loop = _obj(raw, "loop", "config.json", optional=True)
-        start = stop = 0
-        times = 1
-        if loop is not None:
-            start, stop = require_int(loop, "start", minimum=0), require_int(loop, "stop", minimum=0)
-            times = require_int(loop, "times", minimum=1)
-            if not start < stop <= len(layers):
-                raise ConfigError(f"loop: start {start} < stop {stop} <= {len(layers)} layers does not hold")
+        start, stop, times = read_loop(raw, len(layers))
         eos = raw.get("eos_token_id")
         eos = () if eos is None else tuple(eos) if isinstance(eos, (list, tuple)) else (eos,)
         return cls(require_int(raw, "vocab"), require_int(raw, "width"),
@@ -180,13 +163,7 @@ class ZukotarConfig(ModelConfig):
 
     def layer_runs(self) -> list[tuple[int, int | None]]:
         """[(layer, pass number if the run begins a pass of the loop, else None)] in running order."""
-        n = len(self.layers)
-        if not self.has_loop:
-            return [(i, None) for i in range(n)]
-        runs = [(i, None) for i in range(self.loop_start)]
-        for t in range(self.loop_times):
-            runs += [(i, t if i == self.loop_start else None) for i in range(self.loop_start, self.loop_stop)]
-        return runs + [(i, None) for i in range(self.loop_stop, n)]
+        return looped_runs(len(self.layers), self.loop_start, self.loop_stop, self.loop_times)
 
     def to_dict(self) -> dict[str, Any]:
         d: dict[str, Any] = {

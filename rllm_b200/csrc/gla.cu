@@ -4,6 +4,9 @@
 //   alpha_t[k] = sigmoid(z_t[k] + b[k]) ^ (1 / tau)          computed as exp(logsigmoid(.) / tau)   (gla_decay)
 //   S_t[k, v]  = alpha_t[k] * S_(t-1)[k, v] + key_t[k] * value_t[v]
 //   o_t[v]     = sum_k S_t[k, v] * (query_t[k] * qscale)
+// With a bonus b[k] per head (BONUS) a token reads the state before it and its own product times b, not decayed:
+//   o_t[v]     = sum_k (S_(t-1)[k, v] + b[k] * key_t[k] * value_t[v]) * (query_t[k] * qscale)
+//              = sum_k S_(t-1)[k, v] * query_t[k] * qscale  +  value_t[v] * (sum_k query_t[k] * qscale * b[k] * key_t[k])
 // The state S lives in float in a slot per request and is carried from step to step; a step brings any
 // number of tokens of a sequence (a prompt portion or one decoded token).
 //
@@ -18,7 +21,8 @@
 //   (S_start of each chunk, the final state into the slot), pass FINAL runs each chunk again from its
 //   S_start and writes the outputs. Twice the arithmetic, chunks-fold the parallelism; sums are grouped
 //   differently than token by token, within float rounding.
-// gla_finish: one warp per (token, head): o / sqrt(mean(o^2) + eps) * w over vdim, times silu(gate).
+// gla_finish: one warp per (token, head): o / sqrt(mean(o^2) + eps) * w over vdim (w shared by the heads, or each head's
+//   own), times silu(gate).
 #include "common.cuh"
 using namespace rllm;
 
@@ -50,18 +54,19 @@ __device__ __forceinline__ bool find_chunk(const int* cu_q, int num_seqs, int ch
   return false;
 }
 
-template <typename TI, int KP, int MODE>   // KP: state registers a thread, 4 * KP >= dim
+template <typename TI, int KP, int MODE, bool BONUS>   // KP: state registers a thread, 4 * KP >= dim
 __global__ void __launch_bounds__(128)
 gla_scan_kernel(const TI* __restrict__ proj, long long ld, int q_off, int k_off, int v_off,
                 const float* __restrict__ alpha, float qscale, int H, int dim, int vdim,
                 const int* __restrict__ cu_q, int num_seqs, const int* __restrict__ state_slots,
                 float* __restrict__ state, float* __restrict__ out, int chunk, float* __restrict__ chunk_state,
-                float* __restrict__ chunk_decay, int ch) {
+                float* __restrict__ chunk_decay, int ch, const float* __restrict__ bonus) {
   pdl_launch();
   pdl_wait();
   extern __shared__ __align__(16) float staged[];              // queries, keys, decays: [ch][dimp] each
   __shared__ float vs[CH][32];
   __shared__ float part[CH][4][32];
+  __shared__ float own[BONUS ? CH : 1];                        // a token's own share of what it reads, per unit of value
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int h = blockIdx.y, v = blockIdx.z * 32 + lane;
   int seq = blockIdx.x, c = 0, base = 0;
@@ -130,6 +135,13 @@ gla_scan_kernel(const TI* __restrict__ proj, long long ld, int q_off, int k_off,
       vs[cc][j] = vv < vdim ? to_f32(proj[(long long)(c0 + cc) * ld + v_off + h * vdim + vv]) : 0.f;
     }
     __syncthreads();
+    if (BONUS && MODE != LOCAL)
+      for (int cc = warp; cc < n; cc += 4) {                   // (read after the next barrier)
+        float b = 0.f;
+        for (int k = lane; k < dim; k += 32) b = fmaf(qs[cc * dimp + k] * ks[cc * dimp + k], bonus[h * dim + k], b);
+        b = warp_sum(b);
+        if (lane == 0) own[cc] = b;
+      }
     if (vec) {
       // a warp's key channels are a multiple of 4: decays, keys and queries come four at a time
       for (int cc = 0; cc < n; ++cc) {
@@ -142,10 +154,14 @@ gla_scan_kernel(const TI* __restrict__ proj, long long ld, int q_off, int k_off,
         for (int i = 0; i < KP; i += 4) {
           if (i < kp) {
             const float4 a = a4[i >> 2], kk = k4[i >> 2];
+            if (BONUS && MODE != LOCAL) {                      // what the token reads comes before its own update
+              const float4 q = q4[i >> 2];
+              o = fmaf(S[i], q.x, o); o = fmaf(S[i + 1], q.y, o); o = fmaf(S[i + 2], q.z, o); o = fmaf(S[i + 3], q.w, o);
+            }
             S[i] = fmaf(a.x, S[i], kk.x * val); S[i + 1] = fmaf(a.y, S[i + 1], kk.y * val);
             S[i + 2] = fmaf(a.z, S[i + 2], kk.z * val); S[i + 3] = fmaf(a.w, S[i + 3], kk.w * val);
             if (MODE == LOCAL) { A[i] *= a.x; A[i + 1] *= a.y; A[i + 2] *= a.z; A[i + 3] *= a.w; }
-            else {
+            else if (!BONUS) {
               const float4 q = q4[i >> 2];
               o = fmaf(S[i], q.x, o); o = fmaf(S[i + 1], q.y, o); o = fmaf(S[i + 2], q.z, o); o = fmaf(S[i + 3], q.w, o);
             }
@@ -161,9 +177,10 @@ gla_scan_kernel(const TI* __restrict__ proj, long long ld, int q_off, int k_off,
         for (int i = 0; i < KP; ++i) {
           const int k = kbase + i;
           if (i < kp && k < dim) {
+            if (BONUS && MODE != LOCAL) o = fmaf(S[i], qs[cc * dimp + k], o);
             S[i] = fmaf(as[cc * dimp + k], S[i], ks[cc * dimp + k] * val);
             if (MODE == LOCAL) A[i] *= as[cc * dimp + k];
-            else o = fmaf(S[i], qs[cc * dimp + k], o);
+            else if (!BONUS) o = fmaf(S[i], qs[cc * dimp + k], o);
           }
         }
         if (MODE != LOCAL) part[cc][warp][lane] = o;
@@ -174,8 +191,11 @@ gla_scan_kernel(const TI* __restrict__ proj, long long ld, int q_off, int k_off,
       for (int x = threadIdx.x; x < n * 32; x += 128) {
         const int cc = x >> 5, j = x & 31;
         const int vv = blockIdx.z * 32 + j;
-        if (vv < vdim)
-          out[((long long)(c0 + cc) * H + h) * vdim + vv] = ((part[cc][0][j] + part[cc][1][j]) + part[cc][2][j]) + part[cc][3][j];
+        if (vv < vdim) {
+          float o = ((part[cc][0][j] + part[cc][1][j]) + part[cc][2][j]) + part[cc][3][j];
+          if (BONUS) o = fmaf(own[cc], vs[cc][j], o);
+          out[((long long)(c0 + cc) * H + h) * vdim + vv] = o;
+        }
       }
   }
   if (MODE != FINAL && vok && !(MODE == WHOLE && slot < 0)) {
@@ -223,7 +243,7 @@ __global__ void gla_carry_kernel(const int* __restrict__ cu_q, const int* __rest
 
 template <typename TI>
 __global__ void __launch_bounds__(128)
-gla_finish_kernel(const float* __restrict__ o, const float* __restrict__ w, float eps, const TI* __restrict__ proj,
+gla_finish_kernel(const float* __restrict__ o, const float* __restrict__ w, int w_heads, float eps, const TI* __restrict__ proj,
                   long long ld, int g_off, int T, int H, int vdim, TI* __restrict__ out) {
   pdl_launch();
   pdl_wait();
@@ -237,6 +257,7 @@ gla_finish_kernel(const float* __restrict__ o, const float* __restrict__ w, floa
   ss = warp_sum(ss);
   const float r = 1.f / sqrtf(ss / (float)vdim + eps);
   const TI* g = proj + (long long)t * ld + g_off + h * vdim;
+  if (w_heads) w += h * vdim;                    // a weight per head and column
   TI* dst = out + x * vdim;
   for (int i = lane; i < vdim; i += 32) {
     const float gv = to_f32(g[i]);
@@ -244,17 +265,17 @@ gla_finish_kernel(const float* __restrict__ o, const float* __restrict__ w, floa
   }
 }
 
-template <typename TI, int MODE>
+template <typename TI, int MODE, bool BONUS>
 int scan(dim3 grid, cudaStream_t s, const void* proj, long long ld, int q_off, int k_off, int v_off, const float* alpha,
          float qscale, int H, int dim, int vdim, const int* cu_q, int num_seqs, const int* state_slots, float* state,
-         float* out, int chunk, float* chunk_state, float* chunk_decay, int T) {
+         float* out, int chunk, float* chunk_state, float* chunk_decay, int T, const float* bonus) {
   const int kp = (dim + 3) / 4;
   // tokens staged at a time: 16 (8 for wide heads), 2 for steps of single tokens (the room goes to more CTAs an SM)
   const int ch = T <= 2 * num_seqs ? 2 : (dim <= 128 ? CH : CH / 2);
   const size_t smem = (size_t)3 * ch * ((dim + 3) & ~3) * sizeof(float);                             // at most 24 KB
 #define GO(KP)                                                                                                        \
-  return launch_ex(gla_scan_kernel<TI, KP, MODE>, grid, dim3(128), smem, s, 1, (const TI*)proj, ld, q_off, k_off, v_off, \
-                   alpha, qscale, H, dim, vdim, cu_q, num_seqs, state_slots, state, out, chunk, chunk_state, chunk_decay, ch)
+  return launch_ex(gla_scan_kernel<TI, KP, MODE, BONUS>, grid, dim3(128), smem, s, 1, (const TI*)proj, ld, q_off, k_off, v_off, \
+                   alpha, qscale, H, dim, vdim, cu_q, num_seqs, state_slots, state, out, chunk, chunk_state, chunk_decay, ch, bonus)
   if (kp <= 8) GO(8);
   if (kp <= 16) GO(16);
   if (kp <= 32) GO(32);
@@ -274,29 +295,30 @@ RLLM_API int rllm_gla_decay(float* z, const float* bias, int T, int n, float tau
 }
 
 // proj [T, ld] (storage type): queries at q_off, keys at k_off (H x dim each), values at v_off (H x vdim).
-// alpha float [T, H * dim]: the decays. cu_q [S + 1]: row range of each sequence; state_slots [S] (-1: the state
+// alpha float [T, H * dim]: the decays. bonus float [H * dim] or null: the form with a bonus (top of this file). cu_q [S + 1]: row range of each sequence; state_slots [S] (-1: the state
 // starts at zero and is not kept). state float [slots, H, dim, vdim]. out float [T, H, vdim].
 // chunk <= 0: every sequence's rows in one CTA per (head, 32 columns). chunk > 0: the three passes over chunks of
 // that many tokens; chunk_state: float [T / chunk + S, H, dim, vdim], chunk_decay: float [T / chunk + S, H, dim].
 RLLM_API int rllm_gla_scan(int dt, const void* proj, long long ld, int q_off, int k_off, int v_off, const float* alpha,
                            float qscale, int T, int S, int H, int dim, int vdim, const int* cu_q,
                            const int* state_slots, float* state, float* out, int chunk, float* chunk_state,
-                           float* chunk_decay, void* stream) {
+                           float* chunk_decay, const float* bonus, void* stream) {
   if (S <= 0 || T <= 0) return 0;
   if (H <= 0 || dim <= 0 || dim > MAX_DIM || vdim <= 0) return ERR_BAD_SIZE;
   if (H > 65535 || (vdim + 31) / 32 > 65535) return ERR_TOO_LARGE;
   if (dt != DT_F32 && dt != DT_BF16) return ERR_BAD_DTYPE;
   cudaStream_t s = (cudaStream_t)stream;
   const int vb = (vdim + 31) / 32;
-#define SCAN(MODE, GRID)                                                                                            \
-  (dt == DT_F32 ? scan<float, MODE>(GRID, s, proj, ld, q_off, k_off, v_off, alpha, qscale, H, dim, vdim, cu_q, S,   \
-                                    state_slots, state, out, chunk, chunk_state, chunk_decay, T)                    \
-                : scan<bf16, MODE>(GRID, s, proj, ld, q_off, k_off, v_off, alpha, qscale, H, dim, vdim, cu_q, S,    \
-                                   state_slots, state, out, chunk, chunk_state, chunk_decay, T))
+#define SCAN_B(MODE, BONUS, GRID)                                                                                       \
+  (dt == DT_F32 ? scan<float, MODE, BONUS>(GRID, s, proj, ld, q_off, k_off, v_off, alpha, qscale, H, dim, vdim, cu_q, S, \
+                                           state_slots, state, out, chunk, chunk_state, chunk_decay, T, bonus)          \
+                : scan<bf16, MODE, BONUS>(GRID, s, proj, ld, q_off, k_off, v_off, alpha, qscale, H, dim, vdim, cu_q, S,  \
+                                          state_slots, state, out, chunk, chunk_state, chunk_decay, T, bonus))
+#define SCAN(MODE, GRID) (bonus ? SCAN_B(MODE, true, GRID) : SCAN_B(MODE, false, GRID))
   if (chunk <= 0) return SCAN(WHOLE, dim3(S, H, vb));
   if (!chunk_state || !chunk_decay) return ERR_BAD_SIZE;
   const int chunks = T / chunk + S;                                  // at least as many as the sequences have
-  int rc = SCAN(LOCAL, dim3(chunks, H, vb));
+  int rc = SCAN_B(LOCAL, false, dim3(chunks, H, vb));               // what a chunk builds does not depend on the bonus
   if (rc) return rc;
   const int per = dim * vdim;
   rc = launch_ex(gla_carry_kernel, dim3(S, H, (per + 255) / 256), dim3(256), 0, s, 1, cu_q, state_slots, state,
@@ -304,10 +326,11 @@ RLLM_API int rllm_gla_scan(int dt, const void* proj, long long ld, int q_off, in
   if (rc) return rc;
   return SCAN(FINAL, dim3(chunks, H, vb));
 #undef SCAN
+#undef SCAN_B
 }
 
-// o float [T, H, vdim]; w float [vdim]; gate in proj at g_off (H x vdim, storage type); out [T, H * vdim].
-RLLM_API int rllm_gla_finish(int dt, const float* o, const float* w, float eps, const void* proj, long long ld,
+// o float [T, H, vdim]; w float [vdim], or [H * vdim] with w_heads; gate in proj at g_off (H x vdim, storage type); out [T, H * vdim].
+RLLM_API int rllm_gla_finish(int dt, const float* o, const float* w, int w_heads, float eps, const void* proj, long long ld,
                              int g_off, int T, int H, int vdim, void* out, void* stream) {
   if (T <= 0) return 0;
   if (H <= 0 || vdim <= 0) return ERR_BAD_SIZE;
@@ -315,10 +338,10 @@ RLLM_API int rllm_gla_finish(int dt, const float* o, const float* w, float eps, 
   if (blocks > 2147483647LL) return ERR_TOO_LARGE;
   cudaStream_t s = (cudaStream_t)stream;
   if (dt == DT_F32)
-    return launch_ex(gla_finish_kernel<float>, dim3((unsigned)blocks), dim3(128), 0, s, 1, o, w, eps, (const float*)proj,
+    return launch_ex(gla_finish_kernel<float>, dim3((unsigned)blocks), dim3(128), 0, s, 1, o, w, w_heads, eps, (const float*)proj,
                      ld, g_off, T, H, vdim, (float*)out);
   if (dt == DT_BF16)
-    return launch_ex(gla_finish_kernel<bf16>, dim3((unsigned)blocks), dim3(128), 0, s, 1, o, w, eps, (const bf16*)proj, ld,
+    return launch_ex(gla_finish_kernel<bf16>, dim3((unsigned)blocks), dim3(128), 0, s, 1, o, w, w_heads, eps, (const bf16*)proj, ld,
                      g_off, T, H, vdim, (bf16*)out);
   return ERR_BAD_DTYPE;
 }

@@ -3,7 +3,7 @@
 //
 // Two ways to say which rows belong to which problem:
 //   uniform  every problem g (a head) takes all T rows; its A columns start at g * a_gs, its C columns at
-//            g * c_gs, its weights at B + g * b_gs. grid.z = problems.
+//            g * c_gs, its weights at B + g * b_gs. grid.z = problems. The last problem may have fewer columns (N_last).
 //   ragged   problems (experts) own segments of a sorted row list; a table written on the device by the
 //            routing plan names, per tile of rows, the problem, the first sorted row and the row count;
 //            `rows_in[r]` is the A row a sorted row reads (gather), `rows_out[r]` the C row it writes
@@ -12,8 +12,8 @@
 // Every output element is summed over k in ascending order by one thread: a row's result does not depend
 // on where in a list it stands or on what else is in the batch.
 //
-// Epilogues: store (storage type), store float, relu(x)^2 (storage type). Optional per-(row, problem)
-// gate g: the result is multiplied by sigmoid(g) (uniform mode).
+// Epilogues: store (storage type), store float, relu(x)^2 (storage type). Optional gate g, a number per (row, problem)
+// or one per output: the result is multiplied by sigmoid(g) (uniform mode).
 //
 // bfloat16 problems whose rows are 16-byte aligned (K, strides and offsets multiples of 8) run on the
 // tensor cores instead (grouped_gemm_mma_kernel, in a shape for long and one for short row lists):
@@ -39,7 +39,9 @@ struct GroupedArgs {
   const int* rows_in;      // ragged, optional
   const int* rows_out;     // ragged, optional
   const float* row_scale;  // ragged, optional
-  const void* gate; long long gate_ld;   // uniform, optional: gate[r * gate_ld + g]
+  const void* gate; long long gate_ld;   // uniform, optional: gate[r * gate_ld + g], or with gate_cols
+  int gate_cols;                         // gate[r * gate_ld + g * N + n]
+  int G, N_last;                         // uniform: columns of problem G - 1 (0: N)
 };
 
 template <typename TI, int EPI>
@@ -60,6 +62,8 @@ __global__ void __launch_bounds__(256) grouped_gemm_kernel(const GroupedArgs p) 
     g = blockIdx.z; row0 = blockIdx.y * BM; rows = min(BM, p.T - row0);
   }
   const int n0 = blockIdx.x * BN;
+  const int Ng = !p.tiles && p.N_last && g == p.G - 1 ? p.N_last : p.N;
+  if (n0 >= Ng) return;
   const TI* A = (const TI*)p.A + (p.tiles ? 0 : (long long)g * p.a_gs);
   const TI* B = (const TI*)p.B + (long long)g * p.b_gs;
   if (tid < BM) arow[tid] = tid < rows ? (p.rows_in ? p.rows_in[row0 + tid] : row0 + tid) : -1;
@@ -74,7 +78,7 @@ __global__ void __launch_bounds__(256) grouped_gemm_kernel(const GroupedArgs p) 
     for (int j = 0; j < 4; ++j) {
       const int k = k0 + lk + j;
       As[lk + j][lrow] = (am >= 0 && k < p.K) ? to_f32(A[(long long)am * p.lda + k]) : 0.f;
-      Ws[lk + j][lrow] = (wn < p.N && k < p.K) ? to_f32(B[(long long)wn * p.K + k]) : 0.f;
+      Ws[lk + j][lrow] = (wn < Ng && k < p.K) ? to_f32(B[(long long)wn * p.K + k]) : 0.f;
     }
     __syncthreads();
 #pragma unroll
@@ -99,17 +103,18 @@ __global__ void __launch_bounds__(256) grouped_gemm_kernel(const GroupedArgs p) 
     const int r = row0 + m;
     const long long crow = p.rows_out ? p.rows_out[r] : r;
     float f = p.row_scale ? p.row_scale[r] : 1.f;
-    if (p.gate) {
+    if (p.gate && !p.gate_cols) {
       const float gv = to_f32(((const TI*)p.gate)[(long long)r * p.gate_ld + g]);
       f *= 1.f / (1.f + expf(-gv));
     }
 #pragma unroll
     for (int j = 0; j < TN; ++j) {
       const int n = n0 + tx * TN + j;
-      if (n >= p.N) continue;
+      if (n >= Ng) continue;
       float v = acc[i][j];
       if (EPI == GEPI_RELU2) { v = fmaxf(v, 0.f); v = v * v; }
       v *= f;
+      if (p.gate_cols) v *= 1.f / (1.f + expf(-to_f32(((const TI*)p.gate)[(long long)r * p.gate_ld + (long long)g * p.N + n])));
       const long long o = crow * p.ldc + (p.tiles ? 0 : (long long)g * p.c_gs) + n;
       if (EPI == GEPI_STORE_F32) ((float*)p.C)[o] = v;
       else ((TI*)p.C)[o] = from_f32<TI>(v);
@@ -164,6 +169,8 @@ __global__ void __launch_bounds__(C::WM * C::WN * 32, C::CTAS) grouped_gemm_mma_
     g = blockIdx.z; row0 = blockIdx.y * BM_; rows = min(BM_, p.T - row0);
   }
   const int n0 = blockIdx.x * BN_;
+  const int Ng = !p.tiles && p.N_last && g == p.G - 1 ? p.N_last : p.N;
+  if (n0 >= Ng) return;
   const bf16* A = (const bf16*)p.A + (p.tiles ? 0 : (long long)g * p.a_gs);
   const bf16* B = (const bf16*)p.B + (long long)g * p.b_gs;
   for (int r = tid; r < BM_; r += THREADS) arow[r] = r < rows ? (p.rows_in ? p.rows_in[row0 + r] : row0 + r) : -1;
@@ -182,7 +189,7 @@ __global__ void __launch_bounds__(C::WM * C::WN * 32, C::CTAS) grouped_gemm_mma_
 #pragma unroll
     for (int i = 0; i < BN_ * CPR / THREADS; ++i) {
       const int c = tid + i * THREADS, r = c / CPR, k = kb * BK_ + (c % CPR) * 8;
-      const bool in = n0 + r < p.N && k < p.K;
+      const bool in = n0 + r < Ng && k < p.K;
       cp_async16(Bs + (st * BN_ + r) * LDS + (c % CPR) * 8, B + (in ? (long long)(n0 + r) * p.K + k : 0), in ? 16 : 0);
     }
   };
@@ -236,26 +243,31 @@ __global__ void __launch_bounds__(C::WM * C::WN * 32, C::CTAS) grouped_gemm_mma_
       const int r = row0 + m;
       const long long crow = p.rows_out ? p.rows_out[r] : r;
       float f = p.row_scale ? p.row_scale[r] : 1.f;
-      if (p.gate) {
+      if (p.gate && !p.gate_cols) {
         const float gv = to_f32(((const bf16*)p.gate)[(long long)r * p.gate_ld + g]);
         f *= 1.f / (1.f + expf(-gv));
       }
 #pragma unroll
       for (int j = 0; j < NT; ++j) {
         const int n = n0 + wn * NT * 8 + j * 8 + (lane & 3) * 2;
-        if (n >= p.N) continue;
+        if (n >= Ng) continue;
         float v0 = acc[i][j][half * 2], v1 = acc[i][j][half * 2 + 1];
         if (EPI == GEPI_RELU2) { v0 = fmaxf(v0, 0.f); v0 *= v0; v1 = fmaxf(v1, 0.f); v1 *= v1; }
         v0 *= f; v1 *= f;
+        if (p.gate_cols) {
+          const bf16* gp = (const bf16*)p.gate + (long long)r * p.gate_ld + (long long)g * p.N + n;
+          v0 *= 1.f / (1.f + expf(-to_f32(gp[0])));
+          if (n + 1 < Ng) v1 *= 1.f / (1.f + expf(-to_f32(gp[1])));
+        }
         const long long o = crow * p.ldc + (p.tiles ? 0 : (long long)g * p.c_gs) + n;
         if (EPI == GEPI_STORE_F32) {
           float* c = (float*)p.C + o;
-          if (n + 1 < p.N && !(o & 1)) *reinterpret_cast<float2*>(c) = make_float2(v0, v1);
-          else { c[0] = v0; if (n + 1 < p.N) c[1] = v1; }
+          if (n + 1 < Ng && !(o & 1)) *reinterpret_cast<float2*>(c) = make_float2(v0, v1);
+          else { c[0] = v0; if (n + 1 < Ng) c[1] = v1; }
         } else {
           bf16* c = (bf16*)p.C + o;
-          if (n + 1 < p.N && !(o & 1)) *reinterpret_cast<__nv_bfloat162*>(c) = __floats2bfloat162_rn(v0, v1);
-          else { c[0] = __float2bfloat16_rn(v0); if (n + 1 < p.N) c[1] = __float2bfloat16_rn(v1); }
+          if (n + 1 < Ng && !(o & 1)) *reinterpret_cast<__nv_bfloat162*>(c) = __floats2bfloat162_rn(v0, v1);
+          else { c[0] = __float2bfloat16_rn(v0); if (n + 1 < Ng) c[1] = __float2bfloat16_rn(v1); }
         }
       }
     }
@@ -305,14 +317,17 @@ int launch(int epi, const GroupedArgs& p, dim3 grid, cudaStream_t s) {
 }  // namespace
 
 // Uniform problems: A [T, >= G * a_gs] row stride lda; B [G][N, K]; C [T, ...] row stride ldc, problem g at
-// column g * c_gs. gate (optional, storage type): [T, gate_ld], problem g at column g.
+// column g * c_gs. gate (optional, storage type): [T, gate_ld], problem g at column g, or with gate_cols the gate of
+// output n of problem g at column g * N + n. N_last > 0: problem G - 1 has that many columns (at most N).
 RLLM_API int rllm_grouped_gemm_uniform(int dt, int epi, const void* A, long long lda, long long a_gs, const void* B,
                                        long long b_gs, void* C, long long ldc, long long c_gs, int T, int G, int N,
-                                       int K, const void* gate, long long gate_ld, void* stream) {
+                                       int K, const void* gate, long long gate_ld, int gate_cols, int N_last,
+                                       void* stream) {
   if (T <= 0 || G <= 0 || N <= 0) return 0;
-  if (K <= 0) return ERR_BAD_SIZE;
+  if (K <= 0 || N_last < 0 || N_last > N || (gate && N_last)) return ERR_BAD_SIZE;
   if ((T + BM - 1) / BM > 65535 || G > 65535) return ERR_TOO_LARGE;
-  GroupedArgs p = {A, lda, a_gs, B, b_gs, C, ldc, c_gs, T, N, K, nullptr, nullptr, nullptr, nullptr, nullptr, gate, gate_ld};
+  GroupedArgs p = {A, lda, a_gs, B, b_gs, C, ldc, c_gs, T, N, K, nullptr, nullptr, nullptr, nullptr, nullptr, gate, gate_ld,
+                   gate && gate_cols, G, N_last};
   dim3 grid((N + BN - 1) / BN, (T + BM - 1) / BM, G);
   if (dt == DT_BF16 && mma_ok(p) && T <= FewTile::BM)
     return launch_mma<FewTile>(epi, p, dim3((N + FewTile::BN - 1) / FewTile::BN, 1, G), (cudaStream_t)stream);
@@ -340,7 +355,7 @@ RLLM_API int rllm_grouped_gemm_ragged(int dt, int epi, const void* A, long long 
   if (max_tiles <= 0 || N <= 0) return 0;
   if (K <= 0 || !tiles || !n_tiles) return ERR_BAD_SIZE;
   if (max_tiles > 65535) return ERR_TOO_LARGE;
-  GroupedArgs p = {A, lda, 0, B, b_gs, C, ldc, 0, 0, N, K, tiles, n_tiles, rows_in, rows_out, row_scale, nullptr, 0};
+  GroupedArgs p = {A, lda, 0, B, b_gs, C, ldc, 0, 0, N, K, tiles, n_tiles, rows_in, rows_out, row_scale, nullptr, 0, 0, 0, 0};
   dim3 grid((N + BN - 1) / BN, max_tiles, 1);
   if (dt == DT_BF16 && tile_rows == LongTile::BM && mma_ok(p))
     return launch_mma<LongTile>(epi, p, dim3((N + LongTile::BN - 1) / LongTile::BN, max_tiles, 1), (cudaStream_t)stream);

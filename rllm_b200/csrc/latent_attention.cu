@@ -8,7 +8,9 @@
 //
 // latent_prepare (one CTA a token): the latent part of the down-projection is RMS-normed in float
 //   (x / sqrt(mean(x^2) + eps) * w), the shared key part is rotated, and both go to the token's cache
-//   row; the rotated part of every head's query goes to its place behind the folded part in `qfull`.
+//   row; the rotated part of every head's query goes to its place behind the folded part in `qfull`. Queries that
+//   come out of a latent of their own: its norm (`cq`) is part of the first call, which has no queries yet, and
+//   the rotated query parts are a second call without a latent.
 //   Rotation: pairs (2i, 2i+1), i < dims/2, by the angle of the step's table (cos, sin per token and i);
 //   dimensions from `dims` on pass unchanged.
 // latent_attention (one CTA a query token and group of up to 8 heads, a warp a head): keys j with
@@ -29,7 +31,7 @@ __global__ void __launch_bounds__(128)
 latent_prepare_kernel(const TI* __restrict__ proj, long long ld, int q_off, int dkv_off, int H, int dim, int rot,
                       int rank, int dims, const float* __restrict__ wnorm, float eps,
                       const float* __restrict__ table, const int* __restrict__ slots, TI* __restrict__ cache,
-                      TI* __restrict__ qfull) {
+                      TI* __restrict__ qfull, int cq_off, int cq_rank, const float* __restrict__ cq_w, TI* __restrict__ cq) {
   pdl_launch();
   pdl_wait();
   __shared__ float red[32];
@@ -38,12 +40,20 @@ latent_prepare_kernel(const TI* __restrict__ proj, long long ld, int q_off, int 
   const float* tab = table + (long long)t * (dims / 2) * 2;
   const int dk = rank + rot;
   const int slot = slots ? slots[t] : -1;
+  if (cq) {                                      // the queries' latent, normalised
+    float qq = 0.f;
+    for (int i = threadIdx.x; i < cq_rank; i += blockDim.x) { const float v = to_f32(row[cq_off + i]); qq = fmaf(v, v, qq); }
+    qq = block_sum(qq, red);
+    const float rq = 1.f / sqrtf(qq / (float)cq_rank + eps);
+    for (int i = threadIdx.x; i < cq_rank; i += blockDim.x)
+      cq[(long long)t * cq_rank + i] = from_f32<TI>(to_f32(row[cq_off + i]) * rq * cq_w[i]);
+  }
   // the latent, normalised
-  float ss = 0.f;
-  for (int i = threadIdx.x; i < rank; i += blockDim.x) { const float v = to_f32(row[dkv_off + i]); ss = fmaf(v, v, ss); }
-  ss = block_sum(ss, red);
-  const float r = 1.f / sqrtf(ss / (float)rank + eps);
-  if (slot >= 0) {
+  if (slot >= 0) {                               // (the same for the whole CTA)
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < rank; i += blockDim.x) { const float v = to_f32(row[dkv_off + i]); ss = fmaf(v, v, ss); }
+    ss = block_sum(ss, red);
+    const float r = 1.f / sqrtf(ss / (float)rank + eps);
     TI* crow = cache + (long long)slot * dk;
     for (int i = threadIdx.x; i < rank; i += blockDim.x)
       crow[i] = from_f32<TI>(to_f32(row[dkv_off + i]) * r * wnorm[i]);
@@ -60,7 +70,7 @@ latent_prepare_kernel(const TI* __restrict__ proj, long long ld, int q_off, int 
     }
   }
   // every head's rotated query part
-  for (int x = threadIdx.x; x < H * rot; x += blockDim.x) {
+  if (qfull) for (int x = threadIdx.x; x < H * rot; x += blockDim.x) {
     const int h = x / rot, i = x % rot;
     const TI* q = row + q_off + (long long)h * (dim + rot) + dim;
     const float v = to_f32(q[i]);
@@ -620,19 +630,22 @@ latent_merge_kernel(const float* __restrict__ pacc, const float* __restrict__ pm
 // proj [T, ld]: head h's query at q_off + h * (dim + rot) as [dim plain | rot to rotate]; the down-projection
 // at dkv_off as [rank latent | rot shared key part]. table: float [T, dims/2, 2] (cos, sin). slots [T]: cache
 // row of each token (-1: do not write) or null. cache: rows of rank + rot. qfull: [T, H, rank + rot], of which
-// this writes the last rot of every head.
+// this writes the last rot of every head (null: no queries in proj). cq [T, cq_rank] (or null): proj's columns cq_off .. RMS-normed with
+// weight cq_w.
 RLLM_API int rllm_latent_prepare(int dt, const void* proj, long long ld, int q_off, int dkv_off, int T, int H, int dim,
                                  int rot, int rank, int dims, const float* wnorm, float eps, const float* table,
-                                 const int* slots, void* cache, void* qfull, void* stream) {
+                                 const int* slots, void* cache, void* qfull, int cq_off, int cq_rank, const float* cq_w,
+                                 void* cq, void* stream) {
   if (T <= 0) return 0;
   if (H <= 0 || dim < 0 || rot < 0 || rank <= 0 || dims < 0 || dims > rot || dims % 2) return ERR_BAD_SIZE;
+  if ((slots && !wnorm) || (cq && (!cq_w || cq_rank <= 0))) return ERR_BAD_SIZE;
   cudaStream_t s = (cudaStream_t)stream;
   if (dt == DT_F32)
     return launch_ex(latent_prepare_kernel<float>, dim3(T), dim3(128), 0, s, 1, (const float*)proj, ld, q_off, dkv_off, H,
-                     dim, rot, rank, dims, wnorm, eps, table, slots, (float*)cache, (float*)qfull);
+                     dim, rot, rank, dims, wnorm, eps, table, slots, (float*)cache, (float*)qfull, cq_off, cq_rank, cq_w, (float*)cq);
   if (dt == DT_BF16)
     return launch_ex(latent_prepare_kernel<bf16>, dim3(T), dim3(128), 0, s, 1, (const bf16*)proj, ld, q_off, dkv_off, H,
-                     dim, rot, rank, dims, wnorm, eps, table, slots, (bf16*)cache, (bf16*)qfull);
+                     dim, rot, rank, dims, wnorm, eps, table, slots, (bf16*)cache, (bf16*)qfull, cq_off, cq_rank, cq_w, (bf16*)cq);
   return ERR_BAD_DTYPE;
 }
 

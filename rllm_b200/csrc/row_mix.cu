@@ -6,7 +6,8 @@
 //   per-request state; pair_embed_keep writes a portion's last token there afterwards (a kernel of its own: the
 //   slot is read by another CTA of the first).
 // combine: h[t] += sum_i c * w_i * a_i[t] / sqrt(mean(a_i[t]^2) + eps)   (up to two normed summands)
-//                 + sum over up to three plain summands, each [T, parts, H] added in order of parts.
+//                 + sum over up to three plain summands, each [T, parts, H] added in order of parts; the last one
+//                   optionally times the sigmoid of a number per row.
 //   One pass over the row: the sum of a layer's sublayer outputs and the residual sum.
 // glu_act: out[r, f] = act(gate, up) of in[r, f] and in[r, F + f]:
 //   0: silu(g) * u     1: gelu_tanh(g) * u     2: g' = min(g, limit), u' = clamp(u, -limit, limit),
@@ -86,7 +87,8 @@ template <int VEC>
 __global__ void combine_kernel(float* __restrict__ h, const float* __restrict__ n0, const float* __restrict__ w0,
                                const float* __restrict__ n1, const float* __restrict__ w1, float coef, float eps,
                                const float* __restrict__ p0, int parts0, const float* __restrict__ p1, int parts1,
-                               const float* __restrict__ p2, int parts2, int H) {
+                               const float* __restrict__ p2, int parts2, const float* __restrict__ gate2,
+                               long long gate2_ld, int H) {
   pdl_launch();
   pdl_wait();
   struct V { float v[VEC]; };
@@ -99,6 +101,7 @@ __global__ void combine_kernel(float* __restrict__ h, const float* __restrict__ 
   __shared__ float red[32];
   const size_t t = blockIdx.x;
   float r0 = 0.f, r1 = 0.f;
+  const float g2 = gate2 ? 1.f / (1.f + expf(-gate2[t * gate2_ld])) : 1.f;
   if (n0) {
     float ss = 0.f;
     for (int i = threadIdx.x * VEC; i < H; i += blockDim.x * VEC) {
@@ -151,6 +154,10 @@ __global__ void combine_kernel(float* __restrict__ h, const float* __restrict__ 
     for (int e = 0; e < VEC; ++e) f1.v[e] = f2.v[e] = 0.f;
     sum(p1, parts1, f1);
     sum(p2, parts2, f2);
+    if (gate2) {
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) f2.v[e] *= g2;
+    }
     const V hv = ld(h + t * H + i);
     float out[VEC];
 #pragma unroll
@@ -220,8 +227,8 @@ RLLM_API int rllm_pair_embed(const int* ids, const int* positions, const int* to
 }
 
 RLLM_API int rllm_combine(float* h, const float* n0, const float* w0, const float* n1, const float* w1, float coef, float eps,
-                          const float* p0, int parts0, const float* p1, int parts1, const float* p2, int parts2, int T,
-                          int H, void* stream) {
+                          const float* p0, int parts0, const float* p1, int parts1, const float* p2, int parts2,
+                          const float* gate2, long long gate2_ld, int T, int H, void* stream) {
   if (T <= 0) return 0;
   if ((n0 && !w0) || (n1 && !w1)) return ERR_BAD_SIZE;
   const int threads = H >= 1024 ? 256 : 128;
@@ -231,9 +238,9 @@ RLLM_API int rllm_combine(float* h, const float* n0, const float* w0, const floa
     aligned = aligned && (reinterpret_cast<uintptr_t>(q) & 15) == 0;
   if (aligned)
     return launch_ex(combine_kernel<4>, dim3(T), dim3(threads), 0, (cudaStream_t)stream, 1, h, n0, w0, n1, w1, coef, eps, p0,
-                     parts0, p1, parts1, p2, parts2, H);
+                     parts0, p1, parts1, p2, parts2, gate2, gate2_ld, H);
   return launch_ex(combine_kernel<1>, dim3(T), dim3(threads), 0, (cudaStream_t)stream, 1, h, n0, w0, n1, w1, coef, eps, p0, parts0,
-                   p1, parts1, p2, parts2, H);
+                   p1, parts1, p2, parts2, gate2, gate2_ld, H);
 }
 
 RLLM_API int rllm_glu_act(const void* in, int in_dt, long long ld, void* out, int out_dt, int R, int F, int kind, float limit,

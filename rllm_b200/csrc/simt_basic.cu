@@ -36,6 +36,22 @@ RLLM_API int rllm_embed(const int* ids, const void* table, int table_dt, float* 
   return rc;
 }
 
+// ---------------------------------------------------------------- bounded values
+// x <- cap * tanh(x / cap), in place, float (CUDA's tanhf)
+__global__ void softcap_kernel(float* __restrict__ x, long long n, float cap) {
+  pdl_launch();
+  pdl_wait();
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x)
+    x[i] = cap * tanhf(x[i] / cap);
+}
+
+RLLM_API int rllm_softcap(float* x, long long n, float cap, void* stream) {
+  if (n <= 0) return 0;
+  if (!(cap > 0.f)) return ERR_BAD_SIZE;
+  const int blocks = (int)((n + 255) / 256 < 2368 ? (n + 255) / 256 : 2368);
+  return launch_ex(softcap_kernel, dim3(blocks), dim3(256), 0, (cudaStream_t)stream, 1, x, n, cap);
+}
+
 // ---------------------------------------------------------------- a step's metadata onto the device
 // The int32 words of a step's metadata, read straight out of pinned host memory (mapped into the
 // device's address space) into the buffer the step's kernels read. The first n_feed words, the

@@ -81,6 +81,19 @@ class Backend:
         return (w.shape[0] + 127) // 128 <= self._sm100.init(self.device).sm_count or \
             self._sm100.stream_supported(ops.EPI_STORE_F32, True, x.shape[0], w.shape[0], w.shape[1])
 
+    def fuses_norm(self, T):
+        """May a product of a step of T tokens take the norm in front of it into its own kernel?"""
+        return self._sm100 is not None and T <= self._sm100.norm_max_tokens() and os.environ.get("RLLM_B200_NO_NORM_FUSION") != "1"
+
+    def norm_pair(self, h, w, eps, w2, eps2):
+        """Two norms of the same rows in one pass: (h / rms(h) * w, h / rms(h) * w2) in the run dtype; float weights."""
+        _, n, n2 = self._mix.shift_mix(h, w, eps, self.dtype, plain=True, second=(w2, eps2))
+        return n, n2
+
+    def softcap(self, x, cap):
+        """x <- cap * tanh(x / cap), float and in place."""
+        return ops.softcap(x, cap)
+
     def gather_rows(self, x, rows):
         return ops.gather_rows(x, rows)
 
@@ -192,13 +205,35 @@ class Backend:
         """residual += rmsnorm(y) * w (y [T, H], or [T, parts, H] summed over parts first), in float."""
         return self._mix.rmsnorm_add(residual, y, w, eps)
 
-    def add_row(self, h, v):
-        return self._mix.add_row(h, v)
+    def add_row(self, h, v, ids=None, table=None, scale=1.0):
+        """h += v on every row; with token ids and the embedding table, h += table[id] * scale first."""
+        if table is None:
+            return self._mix.add_row(h, v)
+        return self._mix.add_embedding_row(h, v, ids, table, scale)
 
-    def linear_heads(self, a, a_gs, w, out, c_gs, f32=False, gate=None):
-        """One product per head in one launch: out[:, g*c_gs + n] = a[:, g*a_gs : g*a_gs + K] w[g]^T."""
+    def linear_heads(self, a, a_gs, w, out, c_gs, f32=False, gate=None, gate_cols=False):
+        """One product per head in one launch: out[:, g*c_gs + n] = a[:, g*a_gs : g*a_gs + K] w[g]^T, times the sigmoid of
+        a gate per head, or (`gate_cols`) per output."""
         return self._mix.grouped_gemm_uniform(a, a_gs, w, out, c_gs,
-                                              self._mix.GEPI_STORE_F32 if f32 else self._mix.GEPI_STORE, gate=gate)
+                                              self._mix.GEPI_STORE_F32 if f32 else self._mix.GEPI_STORE, gate=gate,
+                                              gate_cols=gate_cols)
+
+    def linear_mixes(self, x, w, rows_each, tag=None):
+        """One product per mix of the input, side by side: out[:, g*N + n] = x[:, g] w[g*N + n]^T with N = rows_each, in the
+        run dtype; x [T, G, K], w [R, K] the problems' rows under each other, the last one with what is left of R. Steps
+        of few tokens run as one launch that streams all weights, longer ones as a tensor-core product each."""
+        T, G, K = x.shape
+        N = int(rows_each)
+        out = torch.empty((T, w.shape[0]), dtype=x.dtype, device=x.device)
+        if self._sm100 is None or T <= 32:
+            return self._mix.grouped_gemm_uniform(x.view(T, G * K), K, w, out, N, self._mix.GEPI_STORE, rows_each=N)
+        for g in range(G):
+            wg, xg, og = w[g * N: (g + 1) * N], x[:, g], out[:, g * N: g * N + N]
+            if self._tc(xg, wg) and self._sm100.out_supported(og):
+                self._sm100.gemm(xg, wg, ops.EPI_STORE, out=og)
+            else:
+                ops.gemm_simt(xg, wg, ops.EPI_STORE, out=og)
+        return out
 
     def expert_tile_rows(self, x, w_up, w_down, n_rows):
         """Rows per tile of a plan that the up and the down product of a routed feed-forward share."""
@@ -206,10 +241,12 @@ class Backend:
         down = self._mix.tile_rows(x.dtype, w_down.shape[2], w_down.shape[2], n_rows)
         return up if up == down else 64         # one of them stays on the CUDA cores: both take its tiles
 
-    def route(self, logits, top, groups=1, keep=1, renorm=False, tile_rows=64, score="softmax", bias=None):
-        """Router logits (plus a float bias per expert) -> the plan of the experts' grouped products (all on the device)."""
-        idx, wt = self._mix.moe_topk(logits, top, groups, keep, renorm, score, bias)
-        return idx, wt, self._mix.moe_plan(idx, wt, logits.shape[1], tile_rows)
+    def route(self, logits, top, groups=1, keep=1, renorm=False, tile_rows=64, score="softmax", bias=None, experts=None,
+              correction=None, group_sum=1, sum_eps=0.0, scale=1.0):
+        """Router logits (plus a float bias per expert) -> the plan of the experts' grouped products (all on the device).
+        `experts`: how many of the logits' columns are experts; the rest as for `mix.moe_topk`."""
+        idx, wt = self._mix.moe_topk(logits, top, groups, keep, renorm, score, bias, experts, correction, group_sum, sum_eps, scale)
+        return idx, wt, self._mix.moe_plan(idx, wt, logits.shape[1] if experts is None else experts, tile_rows)
 
     def _tc_experts(self, a, w, plan):
         """Long row lists in bfloat16 go to the tcgen05 grouped product (RLLM_B200_NO_TC_EXPERTS=1: never)."""
@@ -385,8 +422,18 @@ class Backend:
     def gla_finish(self, *a, **k):
         return self._mix.gla_finish(*a, **k)
 
+    def shift_mix(self, h, w, eps, mu, ctx, prev, second=None):
+        """The mixes of a token's normed row with the one before it in its sequence, [T, len(mu), W] in the run dtype, and
+        the rows of a `second` norm (weight, eps) of the same stream, or None."""
+        mixes, _, n2 = self._mix.shift_mix(h, w, eps, self.dtype, mu, ctx.token_seq, ctx.cu_q, ctx.num_seqs, ctx.state_slots,
+                                           prev, second=second)
+        return mixes, n2
+
+    def lowrank_decay(self, z, w2, bias):
+        return self._mix.lowrank_decay(z, w2, bias)
+
     # ---- recurrent mixers with a short convolution, attention with mixed heads, layers whose sublayers run side by
-    # side (libraries "recurrent" and "hybrid")
+    # side (libraries "recurrent", "rows" and "hybrid")
     @property
     def _hy(self):
         from . import hybrid
@@ -400,8 +447,9 @@ class Backend:
 
     def combine(self, h, *outputs):
         """h += the sublayers' outputs, in float and in one pass. An output is a float tensor [T, H] / [T, parts, H],
-        `Summands` (parts and an ungated second summand) or `NormedSum` (summands that are RMS-normed first)."""
-        normed, plain, coef, eps = [], [], 1.0, 1e-6
+        `Summands` (parts and a second summand, which one of the outputs may gate) or `NormedSum` (summands that are
+        RMS-normed first)."""
+        normed, plain, coef, eps, gate = [], [], 1.0, 1e-6, None
         for y in outputs:
             if y is None:
                 continue
@@ -410,12 +458,15 @@ class Backend:
                     raise ops.KernelError("combine takes the normed summands of one sublayer")
                 normed, coef, eps = list(y.terms), y.coef, y.eps
             elif hasattr(y, "parts"):
-                if y.extra_gate is not None:
-                    raise ops.KernelError("combine takes no gated summand")
+                if gate is not None:
+                    raise ops.KernelError("combine takes one gated summand, the last")
                 plain += [t for t in (y.parts, y.extra) if t is not None]
+                gate = y.extra_gate
             else:
+                if gate is not None:
+                    raise ops.KernelError("combine takes one gated summand, the last")
                 plain.append(y)
-        return self._hy.combine(h, normed, coef, eps, plain)
+        return self._hy.combine(h, normed, coef, eps, plain, gate)
 
     def linear_glu(self, x, w_gate_up, act, limit=0.0, alpha=1.0):
         """act(x Wg^T, x Wu^T) with w_gate_up = [Wg; Wu] in the run dtype; the two products stay float until the

@@ -1,7 +1,7 @@
 """Python face of the libraries "recurrent" (recurrent mixers over a per-request state with a short causal
-convolution in front, csrc/recurrent.cu) and "hybrid": grouped-query attention whose heads' softmax weights are mixed by a
-matrix (csrc/talk_attention.cu), and the row-wise work of layers whose sublayers run side by side on one normed
-input (csrc/row_mix.cu). Every function checks shapes, dtypes and devices and then calls an `extern "C"`
+convolution in front, csrc/recurrent.cu), "rows", the row-wise work of layers whose sublayers run side by side
+(csrc/row_mix.cu), and "hybrid": grouped-query attention whose heads' softmax weights are mixed by a
+matrix (csrc/talk_attention.cu), and a gated recurrence and sublayers gated into the stream (csrc/gated_ops.cu). Every function checks shapes, dtypes and devices and then calls an `extern "C"`
 launcher on torch's current stream; there is no CPU or library path behind them.
 """
 from __future__ import annotations
@@ -24,12 +24,14 @@ ops.register_signatures("recurrent", {
                         c_int, _P, _P, _P, _P, c_int, _P],
     "rllm_gated_norm": [_P, _P, c_int, _LL, _P, c_int, c_float, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P],
 })
-ops.register_signatures("hybrid", {
+ops.register_signatures("rows", {
     "rllm_pair_embed": [_P, _P, _P, _P, _P, _P, _P, _P, c_int, _P, c_float, _P, c_int, c_int, c_int, c_int, c_int, _LL, _LL,
                         _P, _P],
-    "rllm_combine": [_P, _P, _P, _P, _P, c_float, c_float, _P, c_int, _P, c_int, _P, c_int, c_int, c_int, _P],
+    "rllm_combine": [_P, _P, _P, _P, _P, c_float, c_float, _P, c_int, _P, c_int, _P, c_int, _P, _LL, c_int, c_int, _P],
     "rllm_glu_act": [_P, c_int, _LL, _P, c_int, c_int, c_int, c_int, c_float, c_float, c_int, _P],
     "rllm_add_bias_f32": [_P, _P, c_int, c_int, _P],
+})
+ops.register_signatures("hybrid", {
     "rllm_value_norm_store": [c_int, _P, _LL, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, _P, _P, _P, c_int, _P],
     "rllm_talk_attention_simt": [c_int, _P, _LL, _P, _P, _P, _P, _P, _LL, _P, _P, _P, c_int, c_int, c_int, c_int, c_int,
                                  c_int, c_float, c_int, c_int, _P],
@@ -92,7 +94,7 @@ def pair_embed(ids, positions, token_seq, cu_q, num_seqs, state_slots, prev_stat
         _f32(norm_w, "embedding norm weight", (H,))
     out = torch.empty((T, H), dtype=torch.float32, device=table.device)
     keeps = pair is not None and state_slots is not None
-    _check(_fn("hybrid", "rllm_pair_embed")(
+    _check(_fn("rows", "rllm_pair_embed")(
         ids.data_ptr(), positions.data_ptr(), token_seq.data_ptr(), cu_q.data_ptr(), _ptr(state_slots) if keeps else None,
         _ptr(prev_state) if keeps else None, table.data_ptr(), _ptr(pair), _dt(table, "table"), _ptr(norm_w), float(eps),
         out.data_ptr(), T, int(num_seqs), H, V, int(buckets), int(mul_prev), int(mul_cur), _ptr(err), _stream()),
@@ -100,12 +102,21 @@ def pair_embed(ids, positions, token_seq, cu_q, num_seqs, state_slots, prev_stat
     return out
 
 
-def combine(h, normed=(), coef=1.0, eps=1e-6, plain=()) -> torch.Tensor:
+def combine(h, normed=(), coef=1.0, eps=1e-6, plain=(), gate=None) -> torch.Tensor:
     """h (float32 [T, H], in place) += coef * sum_i w_i * a_i / rms(a_i) over `normed` (up to two (a_i, w_i) pairs,
     float32 [T, H] and [H]) + the `plain` summands (up to three float32 tensors [T, H] or [T, parts, H], each summed
-    over parts in order)."""
+    over parts in order). `gate` float32 [T, >= 1]: the last of three plain summands is multiplied by the sigmoid of the
+    row's first number."""
     _f32(h, "h")
     T, H = h.shape
+    gate_ld = 0
+    if gate is not None:
+        _rows(gate, "gate", 1)
+        if gate.dtype != torch.float32 or gate.shape[0] != T:
+            raise KernelError("the gate of a summand must be float32 rows, one per token")
+        gate_ld = gate.stride(0)
+        if len(plain) < 3:                # the gated one is the kernel's third
+            plain = list(plain[:-1]) + [None] * (3 - len(plain)) + [plain[-1]]
     if len(normed) > 2 or len(plain) > 3:
         raise KernelError("combine takes up to two normed and three plain summands")
     n = []
@@ -116,12 +127,15 @@ def combine(h, normed=(), coef=1.0, eps=1e-6, plain=()) -> torch.Tensor:
     n += [None] * (4 - len(n))
     p = []
     for y in plain:
+        if y is None:
+            p += [None, 0]
+            continue
         _f32(y, "summand")
         if y.shape[0] != T or y.shape[-1] != H or y.dim() not in (2, 3):
             raise KernelError(f"a summand must be [T, H] or [T, parts, H], got {list(y.shape)}")
         p += [y.data_ptr(), 1 if y.dim() == 2 else y.shape[1]]
     p += [None, 0] * (3 - len(plain))
-    _check(_fn("hybrid", "rllm_combine")(h.data_ptr(), *n, float(coef), float(eps), *p, T, H, _stream()), "combine")
+    _check(_fn("rows", "rllm_combine")(h.data_ptr(), *n, float(coef), float(eps), *p, _ptr(gate), gate_ld, T, H, _stream()), "combine")
     return h
 
 
@@ -137,7 +151,7 @@ def glu_act(gu, out_dtype, act: str, limit: float = 0.0, alpha: float = 1.0, blo
     if gu.shape[1] != 2 * F:
         raise KernelError("gate/up rows must hold an even number of columns")
     out = torch.empty((R, F), dtype=out_dtype, device=gu.device)
-    _check(_fn("hybrid", "rllm_glu_act")(gu.data_ptr(), _dt(gu, "gate/up"), gu.stride(0), out.data_ptr(), _dt(out, "out"), R, F,
+    _check(_fn("rows", "rllm_glu_act")(gu.data_ptr(), _dt(gu, "gate/up"), gu.stride(0), out.data_ptr(), _dt(out, "out"), R, F,
                                          GLU_ACTS[act], float(limit), float(alpha), int(block or 0), _stream()), "glu_act")
     return out
 
@@ -146,7 +160,7 @@ def add_bias_f32(y, bias) -> torch.Tensor:
     """y float32 [T, N] += bias float32 [N], in place."""
     _f32(y, "y")
     _f32(bias, "bias", (y.shape[1],))
-    _check(_fn("hybrid", "rllm_add_bias_f32")(y.data_ptr(), bias.data_ptr(), y.shape[0], y.shape[1], _stream()), "add_bias_f32")
+    _check(_fn("rows", "rllm_add_bias_f32")(y.data_ptr(), bias.data_ptr(), y.shape[0], y.shape[1], _stream()), "add_bias_f32")
     return y
 
 

@@ -1,5 +1,6 @@
 """Python face of the libraries "mix" (sequence mixers other than grouped-query attention: attention
-over a cache of compressed latents, gated linear attention as a recurrence over per-request state)
+over a cache of compressed latents, gated linear attention as a recurrence over per-request state, what stands in front of a
+recurrence with token shift)
 and "experts" (routed feed-forwards: top-k routing with limited groups, the plan of a grouped product,
 the grouped product itself, and the norm that follows a sublayer). Like `ops`, every function checks shapes,
 dtypes and devices and then calls an `extern "C"` launcher on torch's current stream; there is no
@@ -19,7 +20,7 @@ GEPI_STORE, GEPI_STORE_F32, GEPI_RELU2, GEPI_SILU_GATED = 0, 1, 2, 3
 
 ops.register_signatures("experts", {
     "rllm_grouped_gemm_uniform": [c_int, c_int, _P, _LL, _LL, _P, _LL, _P, _LL, _LL, c_int, c_int, c_int, c_int,
-                                  _P, _LL, _P],
+                                  _P, _LL, c_int, c_int, _P],
     "rllm_grouped_gemm_ragged": [c_int, c_int, _P, _LL, _P, _LL, _P, _LL, c_int, c_int, _P, _P, c_int, c_int, _P, _P, _P,
                                  _P],
     "rllm_grouped_gemm_tile_rows": [c_int, _LL, c_int, c_int],
@@ -27,20 +28,23 @@ ops.register_signatures("experts", {
     "rllm_grouped_gemm_tc": [c_int, _P, _LL, _LL, _P, c_int, c_int, c_int, _P, _LL, _P, _P, c_int, _P, _P, _P, c_int, c_float,
                              c_float, _P],
     "rllm_gather_rows_bf16": [_P, _LL, _P, _P, c_int, c_int, _P],
-    "rllm_moe_topk": [_P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P, _P, _P],
+    "rllm_moe_topk": [_P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P, c_float, c_float, _P, _P, _P],
     "rllm_moe_plan": [_P, _P, c_int, c_int, c_int, c_int, _P, _P, _P, _P, _P, _P],
     "rllm_rmsnorm_add": [_P, c_int, _P, _P, c_int, c_int, c_float, _P],
     "rllm_add_row": [_P, _P, c_int, c_int, _P],
+    "rllm_add_embedding_row": [_P, _P, _P, _P, c_int, c_float, c_int, c_int, c_int, _P],
 })
 ops.register_signatures("mix", {
     "rllm_latent_prepare": [c_int, _P, _LL, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_float, _P,
-                            _P, _P, _P, _P],
+                            _P, _P, _P, c_int, c_int, _P, _P, _P],
     "rllm_latent_attention": [c_int, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
                               c_int, _P, c_int, c_int, c_int, c_int, _P, _P, _P],
     "rllm_gla_decay": [_P, _P, c_int, c_int, c_float, _P],
     "rllm_gla_scan": [c_int, _P, _LL, c_int, c_int, c_int, _P, c_float, c_int, c_int, c_int, c_int, c_int, _P, _P, _P,
-                      _P, c_int, _P, _P, _P],
-    "rllm_gla_finish": [c_int, _P, _P, c_float, _P, _LL, c_int, c_int, c_int, c_int, _P, _P],
+                      _P, c_int, _P, _P, _P, _P],
+    "rllm_shift_mix": [c_int, _P, _P, c_float, _P, c_float, _P, c_int, _P, _P, _P, _P, _P, _P, _P, c_int, c_int, _P],
+    "rllm_lowrank_decay": [c_int, _P, _LL, c_int, _P, _P, _P, c_int, c_int, _P],
+    "rllm_gla_finish": [c_int, _P, _P, c_int, c_float, _P, _LL, c_int, c_int, c_int, c_int, _P, _P],
 })
 
 
@@ -87,29 +91,54 @@ def add_row(h: torch.Tensor, v: torch.Tensor) -> torch.Tensor:
     return h
 
 
+def add_embedding_row(h: torch.Tensor, v: torch.Tensor, ids: torch.Tensor, table: torch.Tensor, scale: float) -> torch.Tensor:
+    """h [T, H] += table[ids[t]] * scale, then += v [H], on every row, float32, in place; table [V, H]."""
+    _f32(h, "h")
+    T, H = h.shape
+    _f32(v, "v", (H,))
+    _i32(ids, "ids", T)
+    _cuda(table, "table")
+    if table.dim() != 2 or not table.is_contiguous() or table.shape[1] != H:
+        raise KernelError(f"the embedding table must be contiguous [V, {H}]")
+    _check(_fn("experts", "rllm_add_embedding_row")(h.data_ptr(), v.data_ptr(), ids.data_ptr(), table.data_ptr(),
+                                                    _dt(table, "table"), float(scale), T, H, table.shape[0], _stream()),
+           "add_embedding_row")
+    return h
+
+
 # --------------------------------------------------------------------------- grouped products
 
 def grouped_gemm_uniform(a: torch.Tensor, a_gs: int, w: torch.Tensor, out: torch.Tensor, c_gs: int, epilogue: int,
-                         gate: torch.Tensor | None = None) -> torch.Tensor:
+                         gate: torch.Tensor | None = None, gate_cols: bool = False, rows_each: int = 0) -> torch.Tensor:
     """out[t, g * c_gs + n] = sum_k a[t, g * a_gs + k] * w[g, n, k] for every problem g (times
-    sigmoid(gate[t, g]) when a gate is given). a [T, >= (G-1) * a_gs + K]; w [G, N, K] contiguous, of a's
-    dtype; out [T, >= (G-1) * c_gs + N] float32 for GEPI_STORE_F32, else of a's dtype; gate [T, >= G] of
-    a's dtype, unit inner stride."""
-    G, N, K = w.shape
+    sigmoid(gate[t, g]) when a gate is given, or sigmoid(gate[t, g * N + n]) with `gate_cols`).
+    a [T, >= (G-1) * a_gs + K]; w [G, N, K] contiguous, of a's dtype; out [T, >= (G-1) * c_gs + N] float32 for
+    GEPI_STORE_F32, else of a's dtype; gate [T, >= G] (G * N) of a's dtype, unit inner stride. `rows_each` = N with
+    w [R, K]: the problems' rows stand under each other, N each, and the last problem has what is left (1 to N)."""
+    if rows_each:
+        N, K = int(rows_each), w.shape[1]
+        G = (w.shape[0] + N - 1) // N
+        last = w.shape[0] - (G - 1) * N
+        if gate is not None:
+            raise KernelError("grouped product: problems of unequal size take no gate")
+    else:
+        G, N, K = w.shape
+        last = N
     _rows(a, "a", (G - 1) * a_gs + K)
-    _rows(out, "out", (G - 1) * c_gs + N)
+    _rows(out, "out", (G - 1) * c_gs + last)
     _cuda(w, "w")
     if not w.is_contiguous() or w.dtype != a.dtype or a.shape[0] != out.shape[0]:
         raise KernelError("grouped product: w must be contiguous [G, N, K] of a's dtype, out must have a's rows")
     if out.dtype != (torch.float32 if epilogue == GEPI_STORE_F32 else a.dtype):
         raise KernelError(f"grouped product: out has dtype {out.dtype}")
     if gate is not None:
-        _rows(gate, "gate", G)
+        _rows(gate, "gate", G * N if gate_cols else G)
         if gate.dtype != a.dtype or gate.shape[0] != a.shape[0]:
             raise KernelError("grouped product: the gate must have a's dtype and rows")
     _check(_fn("experts", "rllm_grouped_gemm_uniform")(
         _dt(a, "a"), epilogue, a.data_ptr(), a.stride(0), a_gs, w.data_ptr(), N * K, out.data_ptr(), out.stride(0),
-        c_gs, a.shape[0], G, N, K, _ptr(gate), 0 if gate is None else gate.stride(0), _stream()), "grouped_gemm_uniform")
+        c_gs, a.shape[0], G, N, K, _ptr(gate), 0 if gate is None else gate.stride(0), int(bool(gate_cols)),
+        0 if last == N else last, _stream()), "grouped_gemm_uniform")
     return out
 
 
@@ -131,21 +160,33 @@ SCORE_FNS = {"softmax": 0, "sigmoid": 1, "softmax_chosen": 2}
 
 
 def moe_topk(logits: torch.Tensor, top: int, groups: int = 1, keep: int = 1,
-             renorm: bool = False, score: str = "softmax", bias: torch.Tensor | None = None) -> tuple[torch.Tensor, torch.Tensor]:
-    """(chosen experts int32 [T, top], their weights float32 [T, top]) from float32 router logits [T, E];
+             renorm: bool = False, score: str = "softmax", bias: torch.Tensor | None = None, experts: int | None = None,
+             correction: torch.Tensor | None = None, group_sum: int = 1, sum_eps: float = 0.0,
+             scale: float = 1.0) -> tuple[torch.Tensor, torch.Tensor]:
+    """(chosen experts int32 [T, top], their weights float32 [T, top]) from float32 router logits [T, E] (or the first
+    `experts` columns of longer rows);
     `score`: "softmax" over all experts, "sigmoid" of each logit by itself, or "softmax_chosen": the logits are
     ranked as they are and the weights are the softmax over the chosen ones only. `bias` float32 [E] is added to
-    the logits first."""
+    the logits first. `correction` float32 [E] is added to the scores for the choice (of groups and experts), not for the
+    weights; `group_sum`: how many of a group's largest scores (1 or 2) make up the group's; `renorm`: weights divided by
+    (their sum + sum_eps); all weights are multiplied by `scale`."""
+    E = logits.shape[1] if experts is None else int(experts)
     if bias is not None:
-        _f32(bias, "router bias", (logits.shape[1],))
+        _f32(bias, "router bias", (E,))
+    if correction is not None:
+        _f32(correction, "router correction", (E,))
     if score not in SCORE_FNS:
         raise KernelError(f"router score {score!r} has no kernel (known: {sorted(SCORE_FNS)})")
-    _f32(logits, "router logits")
-    T, E = logits.shape
+    _rows(logits, "router logits", E)
+    if logits.dtype != torch.float32:
+        raise KernelError("router logits must be float32")
+    T = logits.shape[0]
     idx = torch.empty((T, top), dtype=torch.int32, device=logits.device)
     wt = torch.empty((T, top), dtype=torch.float32, device=logits.device)
-    _check(_fn("experts", "rllm_moe_topk")(logits.data_ptr(), T, E, int(groups), int(keep), int(top), int(bool(renorm)),
-                                           SCORE_FNS[score], ops._ptr(bias), idx.data_ptr(), wt.data_ptr(), _stream()), "moe_topk")
+    _check(_fn("experts", "rllm_moe_topk")(
+        logits.data_ptr(), logits.stride(0), T, E, int(groups), int(keep), int(group_sum), int(top), int(bool(renorm)),
+        SCORE_FNS[score], ops._ptr(bias), ops._ptr(correction), float(sum_eps), float(scale), idx.data_ptr(), wt.data_ptr(),
+        _stream()), "moe_topk")
     return idx, wt
 
 
@@ -239,16 +280,27 @@ def grouped_gemm_tc(a: torch.Tensor, w: torch.Tensor, plan: RoutePlan, out: torc
 # --------------------------------------------------------------------------- attention over latents
 
 def latent_prepare(proj: torch.Tensor, q_off: int, dkv_off: int, heads: int, dim: int, rot: int, rank: int,
-                   dims: int, wnorm: torch.Tensor, eps: float, table: torch.Tensor, slots: torch.Tensor | None,
-                   cache: torch.Tensor | None, qfull: torch.Tensor) -> None:
+                   dims: int, wnorm: torch.Tensor | None, eps: float, table: torch.Tensor, slots: torch.Tensor | None,
+                   cache: torch.Tensor | None, qfull: torch.Tensor | None, cq_off: int = 0,
+                   cq_norm: torch.Tensor | None = None) -> torch.Tensor | None:
     """See csrc/latent_attention.cu. proj [T, cols]; table float32 [T, dims/2, 2]; cache [pages, page,
-    rank + rot] of proj's dtype (None with slots None: nothing is stored); qfull [T, heads, rank + rot]."""
+    rank + rot] of proj's dtype (None with slots None: nothing is stored, proj need hold no latent); qfull
+    [T, heads, rank + rot] (None: proj holds no queries). `cq_norm` float32 [q_rank]: columns cq_off .. of proj RMS-normed
+    with this weight are returned, [T, q_rank] of proj's dtype."""
     T = proj.shape[0]
-    _rows(proj, "proj", max(q_off + heads * (dim + rot), dkv_off + rank + rot))
-    _f32(wnorm, "latent norm weight", (rank,))
+    _rows(proj, "proj", max(q_off + heads * (dim + rot) if qfull is not None else 0,
+                            dkv_off + rank + rot if slots is not None else 0,
+                            cq_off + cq_norm.numel() if cq_norm is not None else 0))
+    if wnorm is not None:
+        _f32(wnorm, "latent norm weight", (rank,))
     _f32(table, "rotation table", (T, dims // 2, 2))
-    _cuda(qfull, "qfull")
-    if qfull.dtype != proj.dtype or tuple(qfull.shape) != (T, heads, rank + rot) or not qfull.is_contiguous():
+    cq = None
+    if cq_norm is not None:
+        _f32(cq_norm, "query latent norm weight")
+        cq = torch.empty((T, cq_norm.numel()), dtype=proj.dtype, device=proj.device)
+    if qfull is not None:
+        _cuda(qfull, "qfull")
+    if qfull is not None and (qfull.dtype != proj.dtype or tuple(qfull.shape) != (T, heads, rank + rot) or not qfull.is_contiguous()):
         raise KernelError(f"qfull must be contiguous [{T}, {heads}, {rank + rot}] of {proj.dtype}")
     if slots is not None:
         _i32(slots, "slots", T)
@@ -257,8 +309,9 @@ def latent_prepare(proj: torch.Tensor, q_off: int, dkv_off: int, heads: int, dim
             raise KernelError(f"the latent cache must be contiguous [pages, page, {rank + rot}] of {proj.dtype}")
     _check(_fn("mix", "rllm_latent_prepare")(
         _dt(proj, "proj"), proj.data_ptr(), proj.stride(0), q_off, dkv_off, T, heads, dim, rot, rank, dims,
-        wnorm.data_ptr(), float(eps), table.data_ptr(), _ptr(slots), _ptr(cache) if slots is not None else None,
-        qfull.data_ptr(), _stream()), "latent_prepare")
+        _ptr(wnorm), float(eps), table.data_ptr(), _ptr(slots), _ptr(cache) if slots is not None else None,
+        _ptr(qfull), int(cq_off), 0 if cq is None else cq.shape[1], _ptr(cq_norm), _ptr(cq), _stream()), "latent_prepare")
+    return cq
 
 
 def latent_attention(qfull: torch.Tensor, cache: torch.Tensor, token_seq: torch.Tensor, positions: torch.Tensor,
@@ -313,8 +366,9 @@ def gla_decay(z: torch.Tensor, bias: torch.Tensor, tau: float) -> torch.Tensor:
 
 def gla_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, alpha: torch.Tensor, qscale: float, heads: int,
              dim: int, vdim: int, cu_q: torch.Tensor, num_seqs: int, state_slots: torch.Tensor | None,
-             state: torch.Tensor, chunk: int = 0) -> torch.Tensor:
+             state: torch.Tensor, chunk: int = 0, bonus: torch.Tensor | None = None) -> torch.Tensor:
     """See csrc/gla.cu. -> float32 [T, heads, vdim]; `state` float32 [slots, heads, dim, vdim] is updated.
+    `bonus` float32 [heads, dim]: a token reads the state before it and its own product times the bonus.
     `chunk` > 0: sequences are cut into chunks of that many tokens that run side by side (long portions)."""
     T = proj.shape[0]
     _rows(proj, "proj", max(q_off + heads * dim, k_off + heads * dim, v_off + heads * vdim))
@@ -325,6 +379,8 @@ def gla_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, alpha: torc
     _i32(cu_q, "cu_q", num_seqs + 1)
     if state_slots is not None:
         _i32(state_slots, "state_slots", num_seqs)
+    if bonus is not None:
+        _f32(bonus, "bonus", (heads, dim))
     out = torch.empty((T, heads, vdim), dtype=torch.float32, device=proj.device)
     cs = cd = None
     if chunk > 0:
@@ -334,18 +390,71 @@ def gla_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, alpha: torc
     _check(_fn("mix", "rllm_gla_scan")(
         _dt(proj, "proj"), proj.data_ptr(), proj.stride(0), q_off, k_off, v_off, alpha.data_ptr(), float(qscale), T,
         num_seqs, heads, dim, vdim, cu_q.data_ptr(), _ptr(state_slots), state.data_ptr(), out.data_ptr(), int(chunk),
-        _ptr(cs), _ptr(cd), _stream()), "gla_scan", 3 if chunk > 0 else 1)
+        _ptr(cs), _ptr(cd), _ptr(bonus), _stream()), "gla_scan", 3 if chunk > 0 else 1)
     return out
 
 
 def gla_finish(o: torch.Tensor, w: torch.Tensor, eps: float, proj: torch.Tensor, g_off: int) -> torch.Tensor:
-    """o float32 [T, heads, vdim] -> [T, heads * vdim] of proj's dtype: per head o / rms(o) * w, times
-    silu of the gate at proj[:, g_off + head * vdim + v]."""
+    """o float32 [T, heads, vdim] -> [T, heads * vdim] of proj's dtype: per head o / rms(o) * w (w float32 [vdim] shared by
+    the heads, or [heads * vdim]), times silu of the gate at proj[:, g_off + head * vdim + v]."""
     _f32(o, "o")
     T, H, vdim = o.shape
-    _f32(w, "w", (vdim,))
+    _f32(w, "w", (vdim,) if w.numel() == vdim else (H * vdim,))
     _rows(proj, "proj", g_off + H * vdim)
     out = torch.empty((T, H * vdim), dtype=proj.dtype, device=proj.device)
-    _check(_fn("mix", "rllm_gla_finish")(_dt(proj, "proj"), o.data_ptr(), w.data_ptr(), float(eps), proj.data_ptr(),
+    _check(_fn("mix", "rllm_gla_finish")(_dt(proj, "proj"), o.data_ptr(), w.data_ptr(), int(w.numel() != vdim), float(eps), proj.data_ptr(),
                                          proj.stride(0), g_off, T, H, vdim, out.data_ptr(), _stream()), "gla_finish")
+    return out
+
+
+# --------------------------------------------------------------------------- in front of a recurrence with token shift
+
+def shift_mix(h: torch.Tensor, w: torch.Tensor, eps: float, out_dtype: torch.dtype, mu: torch.Tensor | None = None,
+              token_seq: torch.Tensor | None = None, cu_q: torch.Tensor | None = None, num_seqs: int = 0,
+              state_slots: torch.Tensor | None = None, prev: torch.Tensor | None = None, plain: bool = False,
+              second: tuple | None = None) -> tuple:
+    """See csrc/time_mix.cu. h float32 [T, W]; w float32 [W]; n = h / rms(h) * w. Returns (mixes, n or None, the second
+    norm's rows or None), all of `out_dtype`: mixes [T, len(mu), W] = n + (n of the row before - n) * mu_m for mu float32
+    [m, W] (None: no mixes), n itself with `plain`, h / rms(h) * w2 for `second` = (w2, eps2). `prev` float32 [slots, W]: the
+    normed row each request's previous portion ended with, read for a portion's first row and updated."""
+    _f32(h, "h")
+    T, W = h.shape
+    _f32(w, "norm weight", (W,))
+    mixes = None
+    if mu is not None:
+        _f32(mu, "mu", (mu.shape[0], W))
+        _i32(token_seq, "token_seq", T)
+        _i32(cu_q, "cu_q", num_seqs + 1)
+        if state_slots is not None:
+            _i32(state_slots, "state_slots", num_seqs)
+            _f32(prev, "previous rows")
+            if prev.dim() != 2 or prev.shape[1] != W:
+                raise KernelError(f"the previous rows must be [slots, {W}], got {list(prev.shape)}")
+        mixes = torch.empty((T, mu.shape[0], W), dtype=out_dtype, device=h.device)
+    out = torch.empty((T, W), dtype=out_dtype, device=h.device) if plain else None
+    out2 = None
+    if second is not None:
+        _f32(second[0], "second norm weight", (W,))
+        out2 = torch.empty((T, W), dtype=out_dtype, device=h.device)
+    shifts = mu is not None
+    keeps = shifts and state_slots is not None
+    _check(_fn("mix", "rllm_shift_mix")(
+        ops._DT[out_dtype], h.data_ptr(), w.data_ptr(), float(eps), _ptr(second[0]) if second is not None else None,
+        float(second[1]) if second is not None else 0.0, _ptr(mu), mu.shape[0] if shifts else 0,
+        _ptr(token_seq) if shifts else None, _ptr(cu_q) if shifts else None, _ptr(state_slots) if keeps else None,
+        _ptr(prev) if keeps else None, _ptr(mixes), _ptr(out), _ptr(out2), T, W, _stream()), "shift_mix")
+    return mixes, out, out2
+
+
+def lowrank_decay(z: torch.Tensor, w2: torch.Tensor, bias: torch.Tensor) -> torch.Tensor:
+    """float32 [T, C]: exp(-exp(w2 tanh(z) + bias)); z [T, rank] (unit inner stride) and w2 [C, rank] of one dtype."""
+    C, rank = w2.shape
+    _rows(z, "z", rank)
+    _cuda(w2, "w2")
+    if z.dtype != w2.dtype or not w2.is_contiguous() or z.shape[1] != rank:
+        raise KernelError(f"lowrank_decay: z must be [T, {rank}] of w2's dtype, w2 contiguous")
+    _f32(bias, "decay bias", (C,))
+    out = torch.empty((z.shape[0], C), dtype=torch.float32, device=z.device)
+    _check(_fn("mix", "rllm_lowrank_decay")(_dt(z, "z"), z.data_ptr(), z.stride(0), rank, w2.data_ptr(), bias.data_ptr(),
+                                            out.data_ptr(), z.shape[0], C, _stream()), "lowrank_decay")
     return out

@@ -32,6 +32,7 @@ _P = c_void_p
 _SIGS = {
     "simt": {
         "rllm_embed": [_P, _P, c_int, _P, c_int, c_int, c_int, _P, c_float, _P],
+        "rllm_softcap": [_P, c_longlong, c_float, _P],
         "rllm_rmsnorm": [_P, _P, _P, c_int, _P, c_int, c_int, c_int, c_float, _P],
         "rllm_rope_table": [_P, _P, _P, c_int, c_int, c_float, _P],
         "rllm_rope_cache_write": [_P, c_int, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int,
@@ -128,6 +129,15 @@ def embed(ids: torch.Tensor, table: torch.Tensor, out: torch.Tensor | None = Non
     _check(_fn("simt", "rllm_embed")(ids.data_ptr(), table.data_ptr(), _dt(table, "table"),
                                      out.data_ptr(), T, H, V, _ptr(err), float(scale), _stream()), "embed")
     return out
+
+
+def softcap(x: torch.Tensor, cap: float) -> torch.Tensor:
+    """x <- cap * tanh(x / cap), element by element and in place, float32."""
+    _cuda(x, "x")
+    if x.dtype != torch.float32 or not x.is_contiguous():
+        raise KernelError("softcap works on contiguous float32 values")
+    _check(_fn("simt", "rllm_softcap")(x.data_ptr(), x.numel(), float(cap), _stream()), "softcap")
+    return x
 
 
 def rmsnorm(x: torch.Tensor, w: torch.Tensor, eps: float, out_dtype: torch.dtype,

@@ -147,10 +147,34 @@ class OpProfile:
     def rmsnorm_add(self, residual, y, w, eps):
         return self._timed("norm+add", _nbytes(y) + 2 * _nbytes(residual), 0, self._be.rmsnorm_add, residual, y, w, eps)
 
-    def linear_heads(self, a, a_gs, w, out, c_gs, f32=False, gate=None):
+    def linear_heads(self, a, a_gs, w, out, c_gs, f32=False, gate=None, gate_cols=False):
         T, (G, N, K) = a.shape[0], w.shape
         return self._timed("heads", _nbytes(w) + T * G * (N + K) * a.element_size(), 2 * T * G * N * K,
-                           self._be.linear_heads, a, a_gs, w, out, c_gs, f32=f32, gate=gate)
+                           self._be.linear_heads, a, a_gs, w, out, c_gs, f32=f32, gate=gate, gate_cols=gate_cols)
+
+    def linear_mixes(self, x, w, rows_each, tag=None):
+        T = x.shape[0]
+        return self._timed(tag or "mixes", _nbytes(w, x) + T * w.shape[0] * x.element_size(), 2 * T * w.shape[0] * w.shape[1],
+                           self._be.linear_mixes, x, w, rows_each)
+
+    def shift_mix(self, h, w, eps, mu, ctx, prev, second=None):
+        n = mu.shape[0] + (second is not None)
+        return self._timed("shift_mix", h.numel() * (4 + n * self._be.dtype.itemsize), 0, self._be.shift_mix, h, w, eps, mu, ctx,
+                           prev, second)
+
+    def norm_pair(self, h, *a):
+        return self._timed("norm", h.numel() * (4 + 2 * self._be.dtype.itemsize), 0, self._be.norm_pair, h, *a)
+
+    def lowrank_decay(self, z, w2, bias):
+        T, (C, rank) = z.shape[0], w2.shape
+        return self._timed("decay", _nbytes(w2) + T * (rank * z.element_size() + 4 * C), 2 * T * C * rank, self._be.lowrank_decay,
+                           z, w2, bias)
+
+    def softcap(self, x, cap):
+        return self._timed("softcap", 2 * _nbytes(x), 0, self._be.softcap, x, cap)
+
+    def add_row(self, h, *a, **k):
+        return self._timed("loop_step", 2 * _nbytes(h), 0, self._be.add_row, h, *a, **k)
 
     def expert_tile_rows(self, *a):
         return self._be.expert_tile_rows(*a)
@@ -228,12 +252,13 @@ class OpProfile:
     def gla_decay(self, z, bias, tau):
         return self._timed("gla_decay", 2 * _nbytes(z), 0, self._be.gla_decay, z, bias, tau)
 
-    def gla_scan(self, proj, q_off, k_off, v_off, alpha, qscale, heads, dim, vdim, cu_q, num_seqs, slots, state, chunk=0):
+    def gla_scan(self, proj, q_off, k_off, v_off, alpha, qscale, heads, dim, vdim, cu_q, num_seqs, slots, state, chunk=0,
+                 bonus=None):
         T = proj.shape[0]
         nbytes = T * heads * (2 * dim + vdim) * proj.element_size() + _nbytes(alpha) + T * heads * vdim * 4 \
             + 2 * num_seqs * heads * dim * vdim * 4
         return self._timed("gla_scan", nbytes, 5 * T * heads * dim * vdim, self._be.gla_scan, proj, q_off, k_off, v_off,
-                           alpha, qscale, heads, dim, vdim, cu_q, num_seqs, slots, state, chunk)
+                           alpha, qscale, heads, dim, vdim, cu_q, num_seqs, slots, state, chunk, bonus)
 
     def gla_finish(self, o, *a, **k):
         return self._timed("gla_finish", 2 * _nbytes(o), 0, self._be.gla_finish, o, *a, **k)
@@ -246,8 +271,11 @@ class OpProfile:
     def combine(self, h, *outputs):
         n = 2
         for y in outputs:
-            n += len(y.terms) if hasattr(y, "terms") else 0 if y is None else 1
-        return self._timed("norm+add", n * _nbytes(h), 0, self._be.combine, h, *outputs)
+            if y is None:
+                continue
+            tensors = [t for t, *_ in y.terms] if hasattr(y, "terms") else [y.parts, y.extra] if hasattr(y, "parts") else [y]
+            n += sum(t.numel() for t in tensors if t is not None) / h.numel()
+        return self._timed("norm+add", int(n * _nbytes(h)), 0, self._be.combine, h, *outputs)
 
     def linear_glu(self, x, w_gate_up, act, limit=0.0, alpha=1.0):
         return self._product("gate_up+act", x, w_gate_up, self._be.linear_glu, x, w_gate_up, act, limit, alpha)

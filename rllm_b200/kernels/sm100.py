@@ -115,6 +115,11 @@ def gemm_supported(x: torch.Tensor, w: torch.Tensor) -> bool:
             and x.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0 and x.shape[0] > 0)
 
 
+def out_supported(out: torch.Tensor) -> bool:
+    """May a product store into these rows (a view into longer ones, say)? They start on 16-byte boundaries."""
+    return out.stride(1) == 1 and out.data_ptr() % 16 == 0 and out.stride(0) * out.element_size() % 16 == 0
+
+
 def plan(epilogue: int, T: int, N: int, K: int, device="cuda:0", split: bool | int = True) -> tuple[int, int]:
     """(token tile, ranges of K = CTAs per cluster) the tcgen05 launcher chooses for a problem.
     `split`: False one CTA per tile, True its own choice, a number > 1 that many ranges."""

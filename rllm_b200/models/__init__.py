@@ -5,5 +5,6 @@ from . import livovik  # registers Livovik
 from . import bazulorn  # registers Bazulorn
 from . import purozen  # registers Purozen
 from . import danonex  # registers Danonex
+from . import zufotar  # registers Zufotar
 
-__all__ = ["LayerCall", "Model", "llama", "zukotar", "livovik", "bazulorn", "purozen", "danonex"]
+__all__ = ["LayerCall", "Model", "llama", "zukotar", "livovik", "bazulorn", "purozen", "danonex", "zufotar"]

@@ -28,6 +28,21 @@ class LayerCall:
         return () if self.cache_layer < 0 else (self.cache_layer,)
 
 
+def looped_schedule(blocks: list[Part], runs, steps: list[Part]) -> list[LayerCall]:
+    """The schedule of layers of which a stretch may run several times: `runs` is [(block, number of the pass that the run
+    begins, or None)], `steps[t]` the block that pass t begins with (appended to `blocks` here). Every run of a
+    layer has a cache layer of its own."""
+    first = len(blocks)
+    blocks += steps
+    schedule, cache_layer = [], 0
+    for i, begins in runs:
+        if begins is not None:
+            schedule.append(LayerCall(first + begins, -1))
+        schedule.append(LayerCall(i, cache_layer, True))
+        cache_layer += 1
+    return schedule
+
+
 class Model:
     def __init__(self, config, embedding: Part, blocks: list[Part], schedule: list[LayerCall],
                  head: Part, prefix: str = "model."):

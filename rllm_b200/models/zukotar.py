@@ -10,7 +10,7 @@ from ..config.base import register_architecture
 from ..config.zukotar import ZukotarConfig
 from ..parts import (Embedding, GatedLinearAttention, InterleavedRotary, LatentAttention, LoopStep, RMSNorm,
                      RoutedExperts, SandwichBlock, make_part)
-from .model import LayerCall, Model
+from .model import Model, looped_schedule
 
 
 def _mixer(cfg: ZukotarConfig, layer):
@@ -46,14 +46,7 @@ def build_zukotar(cfg: ZukotarConfig) -> Model:
             step = LoopStep(W, cfg.loop_times, t, owner=steps[0] if steps else None)
             step.prefix = "loop."
             steps.append(step)
-    first_step = len(blocks)
-    blocks += steps
-    schedule, cache_layer = [], 0
-    for i, begins in cfg.layer_runs():
-        if begins is not None:
-            schedule.append(LayerCall(first_step + begins, -1))
-        schedule.append(LayerCall(i, cache_layer, True))     # every run of a layer has its own cache or state
-        cache_layer += 1
+    schedule = looped_schedule(blocks, cfg.layer_runs(), steps)
     final_norm = RMSNorm(W, eps, "norm")
     final_norm.prefix = "final."
     head = make_part("head", "linear", vocab=cfg.vocab, hidden=W, norm=final_norm, tied_to=emb)

@@ -7,7 +7,7 @@ from .attention import GQAttention, SinkGQAttention, TalkingHeadsAttention
 from .ffn import ActFFN, GluFFN, SwiGLU
 from .block import GatedPreNormBlock, LoopStep, OutputNormBlock, ParallelBlock, PostNormBlock, PreNormBlock, SandwichBlock
 from .latent_attention import LatentAttention, LatentCacheSpec
-from .gla import GatedLinearAttention
+from .gla import GatedLinearAttention, TimeMixing
 from .moe import GatedRoutedExperts, GluRoutedExperts, RoutedExperts
 from .recurrent import DeltaRuleMixer, MinGRUMixer, SideBySideMixer, StateSpaceMixer
 from .embedding import Embedding, OutputHead, PairEmbedding
@@ -20,4 +20,4 @@ __all__ = ["CacheKind", "cache_kind_of", "register_cache_kind", "register_rope_r
            "LatentCacheSpec", "GatedLinearAttention", "RoutedExperts", "Summands", "SinkGQAttention", "ActFFN",
            "PostNormBlock", "GatedRoutedExperts", "NormedSum", "TalkingHeadsAttention", "GluFFN", "ParallelBlock",
            "GluRoutedExperts", "DeltaRuleMixer", "SideBySideMixer", "StateSpaceMixer", "PairEmbedding", "ScaledSum",
-           "GatedPreNormBlock", "MinGRUMixer", "OutputNormBlock"]
+           "GatedPreNormBlock", "MinGRUMixer", "OutputNormBlock", "TimeMixing"]

@@ -2,10 +2,11 @@
 order (src/model/registry/llama.rs:163-245): h += mixer(norm(h)); h += ffn(norm(h)).
 `SandwichBlock` norms each sublayer's output as well: h += norm_b(mixer(norm(h))), the same for
 the feed-forward, which may be absent. `LoopStep` is a block that only adds a learned vector to
-every row: what a pass of a looped stretch of layers begins with. `PostNormBlock` norms after the sum,
+every row, and before it the embedding's output again where it is given the embedding: what a pass of a looped stretch of
+layers begins with. `PostNormBlock` norms after the sum,
 h = norm(alpha h + sublayer(h)), the sublayers reading the stream itself; `OutputNormBlock` norms the sublayer's output
 alone, h += coef * norm(sublayer(h)), the sublayers again reading the stream itself. `ParallelBlock` has one norm whose
-output both sublayers read: h += mixer(n) + ffn(n), n = norm(h). `GatedPreNormBlock` is the pre-norm order with a
+output both sublayers read, or one norm each: h += mixer(n) + ffn(n), n = norm(h), or h += mixer(norm1(h)) + ffn(norm2(h)). `GatedPreNormBlock` is the pre-norm order with a
 gate on each sublayer's way into the stream: h += sigmoid(W_g n + b_g) * sublayer(n), n = norm(h), W_g a square matrix."""
 from __future__ import annotations
 
@@ -173,21 +174,26 @@ class OutputNormBlock(PostNormBlock):
 
 class ParallelBlock(Part):
     """h <- h + (mixer(n) + ffn(n)) with n = norm(h): one norm, both sublayers read its output, the feed-forward may
-    be absent. Sublayers return their float outputs (a tensor, `Summands`, or `NormedSum` for a mixer whose members are
+    be absent. With `ffn_norm` the feed-forward reads a norm of its own of the same h; the two are made in one pass where
+    they are not part of a product's kernel, and a mixer that norms the stream itself (`norms_stream`) makes both. Sublayers return their float outputs (a tensor, `Summands`, or `NormedSum` for a mixer whose members are
     normed before they are added); the sum of all of them and the residual sum are one float kernel. A mixer made
     of several mixers gets a tuple of cache layers. `names`: checkpoint sub-prefixes of mixer and feed-forward; the
     norm's weight is a tensor named by its `weight_name` under the block's prefix."""
     graph_safe = True
 
-    def __init__(self, norm: Part, mixer: Part, ffn: Part | None = None, names=("mix.", "mlp.")):
-        self.norm, self.mixer, self.ffn, self.names = norm, mixer, ffn, names
+    def __init__(self, norm: Part, mixer: Part, ffn: Part | None = None, names=("mix.", "mlp."), ffn_norm: Part | None = None):
+        self.norm, self.mixer, self.ffn, self.names, self.ffn_norm = norm, mixer, ffn, names, ffn_norm
+        if getattr(mixer, "norms_stream", False) and ffn is not None and ffn_norm is None:
+            raise ValueError("a mixer that norms the stream itself leaves no normed rows for the feed-forward")
 
     def children(self):
-        return [p for p in (self.norm, self.mixer, self.ffn) if p is not None]
+        return [p for p in (self.norm, self.ffn_norm, self.mixer, self.ffn) if p is not None]
 
     def set_prefix(self, prefix: str):
         self.prefix = prefix
         self.norm.prefix = prefix
+        if self.ffn_norm is not None:
+            self.ffn_norm.prefix = prefix
         for part, sub in ((self.mixer, self.names[0]), (self.ffn, self.names[1])):
             if part is None:
                 continue
@@ -204,10 +210,26 @@ class ParallelBlock(Part):
 
     def forward(self, h, ctx, cache):
         """h: float32 residual stream [T, hidden], updated in place."""
-        n = self.norm.forward(h, ctx)
-        m = self.mixer.forward(n, ctx, cache, None)
-        f = None if self.ffn is None else self.ffn.forward(n, ctx, None)
-        return ctx.backend.combine(h, m, f)
+        be = ctx.backend
+        if self.ffn_norm is None and not getattr(self.mixer, "norms_stream", False):
+            n = n2 = self.norm.forward(h, ctx)
+            m = self.mixer.forward(n, ctx, cache, None)
+        else:
+            # which norms run inside the first product of their sublayer
+            inside = lambda part: part is not None and getattr(part, "takes_deferred", False) and be.fuses_norm(h.shape[0])
+            n2 = self.ffn_norm.deferred(h, ctx) if inside(self.ffn) else None
+            second = (self.ffn_norm.weight_f32(), self.ffn_norm.eps) if self.ffn is not None and n2 is None else None
+            if getattr(self.mixer, "norms_stream", False):
+                m, made = self.mixer.forward_stream(h, self.norm, ctx, cache, second)
+                n2 = made if second is not None else n2
+            elif second is not None and not inside(self.mixer):
+                n, n2 = be.norm_pair(h, self.norm.weight_f32(), self.norm.eps, *second)
+                m = self.mixer.forward(n, ctx, cache, None)
+            else:
+                n2 = self.ffn_norm.forward(h, ctx) if second is not None else n2
+                m = self.mixer.forward(PreNormBlock._norm(self.norm, self.mixer, h, ctx), ctx, cache, None)
+        f = None if self.ffn is None else self.ffn.forward(n2, ctx, None)
+        return be.combine(h, m, f)
 
 
 class GatedPreNormBlock(Part):
@@ -274,11 +296,14 @@ class GatedPreNormBlock(Part):
 
 class LoopStep(Part):
     """h += table[index] on every row. The passes of one loop share the table [times, hidden]: the
-    first owns the tensor (`owner` None), the others name the first."""
+    first owns the tensor (`owner` None), the others name the first. `embedding`: its output for the step's tokens is added
+    first (looked up again, not kept)."""
     graph_safe = True
 
-    def __init__(self, hidden: int, times: int, index: int, owner: "LoopStep | None" = None, name: str = "step"):
+    def __init__(self, hidden: int, times: int, index: int, owner: "LoopStep | None" = None, name: str = "step",
+                 embedding: Part | None = None):
         self.hidden, self.times, self.index, self.owner, self.name = hidden, times, index, owner, name
+        self.embedding = embedding
         self.table = None
 
     def params(self):
@@ -294,7 +319,9 @@ class LoopStep(Part):
         self._row = table[self.index].float().contiguous()
 
     def forward(self, h, ctx, cache=None):
-        return ctx.backend.add_row(h, self._row)
+        if self.embedding is None:
+            return ctx.backend.add_row(h, self._row)
+        return ctx.backend.add_row(h, self._row, ctx.token_ids, self.embedding.table, self.embedding.scale)
 
 
 register_part("block", "prenorm", PreNormBlock)

@@ -2,7 +2,7 @@
 times `scale` for designs that scale it (1 otherwise; a head tied to the table uses the table itself); the head is final norm, then a product with
 `lm_head.weight`, or with the embedding table when the two are tied
 (src/model/primitives.rs:124-143, 1467; src/model/loader/mod.rs:693-702). Logits are
-float32 and are computed only for the rows that were asked for."""
+float32 and are computed only for the rows that were asked for; `softcap` bounds them, cap * tanh(logits / cap)."""
 from __future__ import annotations
 
 from .base import Param, Part, Source, StateSpec, register_part
@@ -29,8 +29,9 @@ class OutputHead(Part):
     graph_safe = True
 
     def __init__(self, vocab: int, hidden: int, norm: Part, tied_to: Embedding | None,
-                 name: str = "weight"):
+                 name: str = "weight", softcap: float | None = None):
         self.vocab, self.hidden, self.norm, self.tied_to, self.name = vocab, hidden, norm, tied_to, name
+        self.softcap = softcap
         self.weight = None
 
     def children(self):
@@ -50,7 +51,8 @@ class OutputHead(Part):
             n = self.norm.deferred(h, ctx, rows)      # gather, norm and product may be one kernel
         else:
             n = self.norm.forward(ctx.backend.gather_rows(h, rows), ctx)
-        return ctx.backend.linear_f32(n, self.matrix())
+        logits = ctx.backend.linear_f32(n, self.matrix())
+        return logits if self.softcap is None else ctx.backend.softcap(logits, self.softcap)
 
 
 register_part("embedding", "table", Embedding)

@@ -36,6 +36,7 @@ class ActFFN(Part):
     """down(act(up x)), no biases; act: "relu2" = max(., 0)^2, "gelu_tanh" = 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))),
     "gelu_erf" = 0.5 z (1 + erf(z / sqrt 2))."""
     graph_safe = True
+    takes_deferred = True
     returns_output = True
     ACTS = ("relu2", "gelu_tanh", "gelu_erf")
 

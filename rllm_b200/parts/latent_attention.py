@@ -9,8 +9,10 @@ values alike). The up-projections never run over the cache: with
 W_uk is folded into the query before the attention kernel and W_uv applied to its output, both as
 one product per head in one launch. Scores are (plain + rotated part) * `scale`, softmax over the keys
 a `window` allows (None: all earlier ones); each head's output is multiplied by sigmoid of a gate
-projected from h (`gate` False: there is none); W_o follows. `rot_dim` 0 with `position` None: no rotated part,
-positions do not enter the scores. Scores, softmax, the latent's norm and the rotation are float.
+projected from h, one number per head (`gate` "head", or True), or one per output of every head (`gate` "full"; False:
+there is none); W_o follows. `q_rank`: the queries come out of a latent of their own, q = W_uq RMSnorm(W_dq h). `rot_dim` 0
+with `position` None: no rotated part, positions do not enter the scores. Scores, softmax, the latents' norms and the
+rotation are float.
 """
 from __future__ import annotations
 
@@ -43,21 +45,28 @@ class LatentAttention(Part):
     returns_output = True      # forward(..., residual=None) returns the float output instead of adding it
 
     def __init__(self, hidden: int, heads: int, dim: int, rot_dim: int, vdim: int, kv_rank: int, scale: float,
-                 position: Part | None, window: int | None = None, eps: float = 1e-6, gate: bool = True):
+                 position: Part | None, window: int | None = None, eps: float = 1e-6, gate: bool | str = True,
+                 q_rank: int | None = None):
         if (position is None) != (rot_dim == 0):
             raise ValueError("a rotated part needs a position part, and only a rotated part does")
         self.hidden, self.heads, self.dim, self.rot_dim, self.vdim = hidden, heads, dim, rot_dim, vdim
         self.kv_rank, self.scale, self.position, self.window, self.eps = kv_rank, float(scale), position, window, float(eps)
-        self.gate = gate
-        self.w_in = self.w_latent_norm = self.w_uk = self.w_uv = self.w_o = None
+        if gate not in (True, False, "head", "full"):
+            raise ValueError(f"output gate {gate!r} is not known (known: 'head', 'full', False)")
+        self.gate = "head" if gate is True else gate or None
+        self.q_rank = q_rank
+        self.w_in = self.w_latent_norm = self.w_uk = self.w_uv = self.w_o = self.w_q_norm = self.w_uq = None
 
     def children(self):
         return [] if self.position is None else [self.position]
 
     def params(self):
-        H, W = self.heads, self.hidden
-        return [Param("w_in", (Source("q", (H * (self.dim + self.rot_dim), W)),
-                               Source("dkv", (self.kv_rank + self.rot_dim, W))) + ((Source("g", (H, W)),) if self.gate else ())),
+        H, W, QD = self.heads, self.hidden, self.heads * (self.dim + self.rot_dim)
+        gate = {None: (), "head": (Source("g", (H, W)),), "full": (Source("g", (H * self.vdim, W)),)}[self.gate]
+        first = Source("q", (QD, W)) if self.q_rank is None else Source("dq", (self.q_rank, W))
+        own = [] if self.q_rank is None else [Param("w_q_norm", (Source("dq.norm", (self.q_rank,), init="norm"),), role="vector"),
+                                              Param("w_uq", (Source("uq", (QD, self.q_rank)),))]
+        return [Param("w_in", (first, Source("dkv", (self.kv_rank + self.rot_dim, W))) + gate), *own,
                 Param("w_latent_norm", (Source("dkv.norm", (self.kv_rank,), init="norm"),), role="vector"),
                 Param("w_uk", (Source("uk", (H * self.dim, self.kv_rank)),)),
                 Param("w_uv", (Source("uv", (H * self.vdim, self.kv_rank)),)),
@@ -72,12 +81,13 @@ class LatentAttention(Part):
         self._uk_t = self.w_uk.view(H, self.dim, self.kv_rank).transpose(1, 2).contiguous()
         self._uv = self.w_uv.view(H, self.vdim, self.kv_rank)
         self._norm_f32 = self.w_latent_norm.float().contiguous()
+        self._q_norm_f32 = None if self.w_q_norm is None else self.w_q_norm.float().contiguous()
 
     def forward(self, x, ctx, cache, residual=None):
         be = ctx.backend
         H, dk = self.heads, self.kv_rank + self.rot_dim
-        q_cols = H * (self.dim + self.rot_dim)
-        proj = be.linear(x, self.w_in)                                   # [T, q | dkv | gate]
+        q_cols = H * (self.dim + self.rot_dim) if self.q_rank is None else self.q_rank
+        proj = be.linear(x, self.w_in, tag="in")                         # [T, q or its latent | dkv | gate]
         T = proj.shape[0]
         qfull = torch.empty((T, H, dk), dtype=proj.dtype, device=proj.device)
         if self.position is None:
@@ -85,16 +95,24 @@ class LatentAttention(Part):
         else:
             table, dims = self.position.table(ctx), self.position.dims
         writes = cache.writes
-        be.latent_prepare(proj, 0, q_cols, H, self.dim, self.rot_dim, self.kv_rank, dims,
-                          self._norm_f32, self.eps, table, cache.slots if writes else None,
-                          cache.tensors["kv"] if writes else None, qfull)
-        be.linear_heads(proj, self.dim + self.rot_dim, self._uk_t, qfull.view(T, H * dk), dk)
+        stored = (cache.slots, cache.tensors["kv"]) if writes else (None, None)
+        if self.q_rank is None:
+            q = proj
+            be.latent_prepare(proj, 0, q_cols, H, self.dim, self.rot_dim, self.kv_rank, dims, self._norm_f32, self.eps, table,
+                              *stored, qfull)
+        else:
+            cq = be.latent_prepare(proj, 0, q_cols, H, self.dim, self.rot_dim, self.kv_rank, dims, self._norm_f32, self.eps,
+                                   table, *stored, None, cq_off=0, cq_norm=self._q_norm_f32)
+            q = be.linear(cq, self.w_uq, tag="uq")
+            if self.rot_dim:
+                be.latent_prepare(q, 0, 0, H, self.dim, self.rot_dim, self.kv_rank, dims, None, self.eps, table, None, None, qfull)
+        be.linear_heads(q, self.dim + self.rot_dim, self._uk_t, qfull.view(T, H * dk), dk)
         o = be.latent_attention(qfull, cache, ctx, self.kv_rank, self.scale, self.window)
         att = torch.empty((T, H * self.vdim), dtype=proj.dtype, device=proj.device)
         be.linear_heads(o.view(T, H * self.kv_rank), self.kv_rank, self._uv, att, self.vdim,
-                        gate=proj[:, q_cols + dk:] if self.gate else None)
+                        gate=proj[:, q_cols + dk:] if self.gate else None, gate_cols=self.gate == "full")
         if residual is None:
-            return be.linear_f32(att, self.w_o)
+            return be.linear_f32(att, self.w_o, tag="o")
         be.linear_residual(att, self.w_o, residual)
         return None
 

@@ -121,20 +121,30 @@ class GluRoutedExperts(Part):
     W_up h) without biases, act one of `GluFFN.ACTS` with its `limit` and `alpha`. Router logits z = W_router h
     (+ a bias per expert, tensor `router.b`) in float; `score` "softmax_chosen": the `top` largest logits are chosen
     and their weights are the softmax over the chosen logits only ("softmax" and "sigmoid" as for the other routed
-    feed-forwards). `shared`: a dense feed-forward every token uses (its tensors under `shared.`), added as it is.
-    Returns `Summands`: one float row per (token, chosen expert) and the shared expert's output; the block adds them."""
+    feed-forwards). `correction`: a number per expert (tensor `correction`) added to the scores for the choice alone.
+    `groups`, `keep`, `group_sum`: experts form `groups` equal groups of neighbours, a group's score is the sum of its
+    `group_sum` (1 or 2) largest choice scores, only experts of the best `keep` groups can be chosen. `renorm`: weights
+    divided by (their sum + `sum_eps`); `weight_scale` multiplies all weights. `shared`: a dense feed-forward every token
+    uses (its tensors under `shared.`), added as it is, or times sigmoid(W_sg h) (`shared.sg`, one row) with `shared_gate`;
+    that row then stands under the router's in one product. Returns `Summands`: one float row per (token, chosen expert) and the shared expert's output; the block adds them."""
     graph_safe = True
     returns_output = True
 
     def __init__(self, hidden: int, ff: int, experts: int, top: int, act: str = "silu", limit: float = 0.0,
                  alpha: float = 1.0, score: str = "softmax_chosen", renorm: bool = False, router_bias: bool = False,
-                 shared: Part | None = None):
+                 shared: Part | None = None, shared_gate: bool = False, correction: bool = False, groups: int = 1,
+                 keep: int = 1, group_sum: int = 1, sum_eps: float = 0.0, weight_scale: float = 1.0):
         if top > experts:
             raise ValueError(f"top {top} exceeds the {experts} experts")
+        if experts % groups or not 1 <= keep <= groups or top > experts // groups * keep:
+            raise ValueError(f"{experts} experts in {groups} groups of which {keep} are kept do not give {top} experts")
+        self.shared_gate, self.correction = shared_gate and shared is not None, correction
+        self.groups, self.keep, self.group_sum = groups, keep, group_sum
+        self.sum_eps, self.weight_scale = float(sum_eps), float(weight_scale)
         self.hidden, self.ff, self.experts, self.top = hidden, ff, experts, top
         self.act, self.limit, self.alpha = act, float(limit), float(alpha)
         self.score, self.renorm, self.router_bias, self.shared = score, renorm, router_bias, shared
-        self.w_router = self.b_router = self.w_gate_up = self.w_down = None
+        self.w_router = self.b_router = self.v_correction = self.w_gate_up = self.w_down = None
 
     def children(self):
         return [] if self.shared is None else [self.shared]
@@ -146,11 +156,13 @@ class GluRoutedExperts(Part):
 
     def params(self):
         E, W, F = self.experts, self.hidden, self.ff
-        ps = [Param("w_router", (Source("router", (E, W)),)),
+        ps = [Param("w_router", (Source("router", (E, W)),) + ((Source("shared.sg", (1, W)),) if self.shared_gate else ())),
               Param("w_gate_up", tuple(Source(f"e{e}.{n}", (F, W)) for e in range(E) for n in ("gate", "up"))),
               Param("w_down", tuple(Source(f"e{e}.down", (W, F)) for e in range(E)))]
         if self.router_bias:
             ps.append(Param("b_router", (Source("router.b", (E,)),), role="vector"))
+        if self.correction:
+            ps.append(Param("v_correction", (Source("correction", (E,)),), role="vector"))
         return ps
 
     def finalize(self, device, dtype):
@@ -164,6 +176,12 @@ class GluRoutedExperts(Part):
         self._gate_up = self.w_gate_up.view(E, 2 * F, W)
         self._down = self.w_down.view(E, W, F)
         self._bias = None if self.b_router is None else self.b_router.float().contiguous()
+        self._correction = None if self.v_correction is None else self.v_correction.float().contiguous()
+        if self.shared_gate and self.w_router.shape[0] % 16:
+            # router rows and the shared expert's gate row: made up with rows of zeros to a height every product takes
+            padded = self.w_router.new_zeros(((E + 1 + 15) // 16 * 16, W))
+            padded[: E + 1] = self.w_router
+            self.w_router = padded
 
     def forward(self, x, ctx, residual=None):
         if residual is not None:
@@ -171,11 +189,17 @@ class GluRoutedExperts(Part):
         be = ctx.backend
         x = x.tensor() if hasattr(x, "tensor") else x
         T = x.shape[0]
-        _, _, plan = be.route(be.linear_f32(x, self.w_router, tag="router"), self.top, renorm=self.renorm, score=self.score,
-                              bias=self._bias, tile_rows=be.expert_tile_rows(x, self._gate_up, self._down, T * self.top))
+        logits = be.linear_f32(x, self.w_router, tag="router")           # [T, >= experts (+ the shared expert's gate)]
+        _, _, plan = be.route(logits, self.top, self.groups, self.keep, renorm=self.renorm, score=self.score,
+                              bias=self._bias, tile_rows=be.expert_tile_rows(x, self._gate_up, self._down, T * self.top),
+                              experts=self.experts, correction=self._correction, group_sum=self.group_sum,
+                              sum_eps=self.sum_eps, scale=self.weight_scale)
         act = be.experts_glu_up(x, self._gate_up, plan, self.act, self.limit, self.alpha, self._block)
         parts = be.experts_down(act, self._down, plan, T, self.top, scale=True)
-        return Summands(parts, None if self.shared is None else self.shared.forward(x, ctx, None))
+        if self.shared is None:
+            return Summands(parts)
+        return Summands(parts, self.shared.forward(x, ctx, None),
+                        logits[:, self.experts: self.experts + 1] if self.shared_gate else None)
 
 
 register_part("ffn", "moe_glu", GluRoutedExperts)
