@@ -232,12 +232,30 @@ def _danonex_sizes():
     return out
 
 
-BESIDE = {"bazulorn": "zukotar", "purozen": "bazulorn", "danonex": "bazulorn"}       # the design timed beside each one; Llama layers otherwise
+def _zufotar_sizes():
+    """Four layers in the order of the Zukotar model beside them (latent attention, recurrence, recurrence, latent
+    attention), of equal width, heads, latent size, rotated part and experts, with a shared expert of one expert's size, a
+    latent of three times the kv latent's size for the queries and 64 numbers between the decays' two projections; no
+    loop on either side."""
+    zk, out = design_sizes("zukotar"), {}
+    for name, W, H, E, top, ff, G, keep in (("w2048", 2048, 16, 16, 6, 2048, 4, 2), ("w4096", 4096, 32, 32, 8, 2688, 8, 4)):
+        moe = {"kind": "moe", "expert": {"ff": ff}, "shared": {"ff": ff},
+               "router": {"experts": E, "top": top, "groups": {"count": G, "keep": keep}, "scale": 2.5}}
+        att = {"type": "latent_attention", "mlp": moe, "mixer": {
+            "heads": H, "dim": 128, "rot_dim": 64, "vdim": 128, "q_rank": 1536, "kv_rank": 512, "scale": 192 ** -0.5,
+            "rot": {"base": 10000.0, "dims": 64, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}}
+        rec = {"type": "wkv", "mlp": moe, "mixer": {"heads": H, "dim": 128, "decay_rank": 64}}
+        out[name] = ({"architecture": "Zufotar", "vocab": 32000, "width": W, "embedding": {"scale": 1.0}, "norm": {"eps": 1e-6},
+                      "logit_softcap": 30.0, "layers": [att, rec, rec, att]}, zk[name][0])
+    return out
+
+
+BESIDE = {"bazulorn": "zukotar", "purozen": "bazulorn", "danonex": "bazulorn", "zufotar": "zukotar"}       # the design timed beside each one; Llama layers otherwise
 
 
 def design_sizes(design):
     """name -> (the design's configuration, the layers beside it: Llama layers of equal width, depth and active
-    feed-forward weights, for Bazulorn the Zukotar model of equal width, depth, heads and experts, for Purozen and
+    feed-forward weights, for Bazulorn and Zufotar the Zukotar model of equal width, depth, heads and experts, for Purozen and
     Danonex Bazulorn layers of equal width, depth and heads)."""
     if design == "livovik":
         return _livovik_sizes()
@@ -245,6 +263,8 @@ def design_sizes(design):
         return _purozen_sizes()
     if design == "danonex":
         return _danonex_sizes()
+    if design == "zufotar":
+        return _zufotar_sizes()
     if design == "bazulorn":
         zk = design_sizes("zukotar")
         return {name: (cfg, zk[name][0]) for name, cfg in _bazulorn_sizes().items()}
@@ -346,9 +366,9 @@ def main():
     ap.add_argument("--workloads", default="", help="comma-separated: mixed_3b, continuous_8b, or all")
     ap.add_argument("--phase", default="all", choices=["all", "prefill", "decode"],
                     help="run one part only (for profiling; the JSON line then lacks the other parts)")
-    ap.add_argument("--designs", default="", choices=["", "zukotar", "livovik", "bazulorn", "purozen", "danonex"],
+    ap.add_argument("--designs", default="", choices=["", "zukotar", "livovik", "bazulorn", "purozen", "danonex", "zufotar"],
                     help="instead of the default workload: prefill and decode of this design beside Llama layers of "
-                         "equal size (bazulorn: beside Zukotar layers; purozen, danonex: beside Bazulorn layers), random weights, "
+                         "equal size (bazulorn, zufotar: beside Zukotar layers; purozen, danonex: beside Bazulorn layers), random weights, "
                          "with the time per operation; "
                          "prints its own JSON line")
     ap.add_argument("--profile-range", action="store_true",

@@ -256,8 +256,11 @@ __global__ void __launch_bounds__(C::WM * C::WN * 32, C::CTAS) grouped_gemm_mma_
         v0 *= f; v1 *= f;
         if (p.gate_cols) {
           const bf16* gp = (const bf16*)p.gate + (long long)r * p.gate_ld + (long long)g * p.N + n;
-          v0 *= 1.f / (1.f + expf(-to_f32(gp[0])));
-          if (n + 1 < Ng) v1 *= 1.f / (1.f + expf(-to_f32(gp[1])));
+          float2 gv;
+          if (!((uintptr_t)gp & 3) && n + 1 < Ng) gv = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(gp));
+          else gv = make_float2(to_f32(gp[0]), n + 1 < Ng ? to_f32(gp[1]) : 0.f);
+          v0 *= __fdividef(1.f, 1.f + __expf(-gv.x));                  // (rounded to 16 bits below)
+          v1 *= __fdividef(1.f, 1.f + __expf(-gv.y));
         }
         const long long o = crow * p.ldc + (p.tiles ? 0 : (long long)g * p.c_gs) + n;
         if (EPI == GEPI_STORE_F32) {
@@ -329,8 +332,9 @@ RLLM_API int rllm_grouped_gemm_uniform(int dt, int epi, const void* A, long long
   GroupedArgs p = {A, lda, a_gs, B, b_gs, C, ldc, c_gs, T, N, K, nullptr, nullptr, nullptr, nullptr, nullptr, gate, gate_ld,
                    gate && gate_cols, G, N_last};
   dim3 grid((N + BN - 1) / BN, (T + BM - 1) / BM, G);
-  if (dt == DT_BF16 && mma_ok(p) && T <= FewTile::BM)
-    return launch_mma<FewTile>(epi, p, dim3((N + FewTile::BN - 1) / FewTile::BN, 1, G), (cudaStream_t)stream);
+  if (dt == DT_BF16 && mma_ok(p) && T <= 2 * FewTile::BM)          // two row tiles read the weights a second time, from L2
+    return launch_mma<FewTile>(epi, p, dim3((N + FewTile::BN - 1) / FewTile::BN, (T + FewTile::BM - 1) / FewTile::BM, G),
+                               (cudaStream_t)stream);
   if (dt == DT_BF16 && mma_ok(p) && (T + LongTile::BM - 1) / LongTile::BM <= 65535)
     return launch_mma<LongTile>(epi, p, dim3((N + LongTile::BN - 1) / LongTile::BN, (T + LongTile::BM - 1) / LongTile::BM, G),
                                 (cudaStream_t)stream);

@@ -17,7 +17,7 @@
 //
 // The token operand is small and the same for every job, so a warp builds its fragments once,
 // after the predecessor has finished, and keeps them in registers (K up to 8,192), or fetches them
-// chunk by chunk, one chunk ahead (longer K). With RMSNorm in front the fragments are
+// chunk by chunk, one chunk ahead (longer K, and products of several operands side by side). With RMSNorm in front the fragments are
 // bf16(h * g) built from the float residual stream, the warps add up h^2 on the way and the
 // epilogue multiplies by rsqrt(mean + eps), as the tcgen05 kernel does.
 //
@@ -70,6 +70,7 @@ struct Params {
   int up_row0;              // SwiGLU: first weight row of the up half
   const bf16* x;            // token operand [T][K], row stride ldx (NORM: unused)
   long long ldx;
+  int x_rows; long long x_gs;   // x_rows > 0: weight rows in groups of that many (a multiple of 16), group g reads x + g * x_gs
   const float* h;           // NORM: float rows, stride ldh; row of token t = rows ? rows[t] : t
   long long ldh;
   const int* rows;
@@ -122,7 +123,7 @@ __device__ __forceinline__ int tile_row0(const Params& p, int job, int tile) {
 // This lane's token fragment for one chunk: token g, k = k0 + 32 kb + 8 t .. + 7 for kb = 0..3
 // (zeros beyond T or K). NORM: bf16(h * g); the squares of h are added to `ss`.
 template <bool NORM>
-__device__ __forceinline__ void load_frag(const Params& p, int k0, int g, int t, uint4 (&b)[4], float& ss) {
+__device__ __forceinline__ void load_frag(const Params& p, int k0, int g, int t, uint4 (&b)[4], float& ss, long long xoff = 0) {
 #pragma unroll
   for (int kb = 0; kb < 4; ++kb) {
     const int k = k0 + 32 * kb + 8 * t;
@@ -149,7 +150,7 @@ __device__ __forceinline__ void load_frag(const Params& p, int k0, int g, int t,
         b[kb].x = pack2(a.x * gv[0], a.y * gv[1]); b[kb].y = pack2(a.z * gv[2], a.w * gv[3]);
         b[kb].z = pack2(c.x * gv[4], c.y * gv[5]); b[kb].w = pack2(c.z * gv[6], c.w * gv[7]);
       } else {
-        b[kb] = __ldcg(reinterpret_cast<const uint4*>(p.x + (size_t)g * p.ldx + k));
+        b[kb] = __ldcg(reinterpret_cast<const uint4*>(p.x + (size_t)g * p.ldx + xoff + k));
       }
     }
   }
@@ -239,6 +240,15 @@ stream_gemm_kernel(const Params p) {
     __syncwarp();                                // every lane has read the slot that is refilled now
     produce();
   };
+  // which columns of x the slabs of this CTA's job number j read
+  auto x_offset = [&](int j) -> long long {
+    return p.x_rows ? (long long)((blockIdx.x + j * gridDim.x) * 16 / p.x_rows) * p.x_gs : 0;
+  };
+  uint4 bcur[4], bnext[4];                       // NCH 0 only
+  if (!NCH && my_jobs > 0) {
+    float unused = 0.f;
+    load_frag<false>(p, (warp * nchw) * CK, g, t, bcur, unused, x_offset(0));
+  }
   for (int batch0 = 0; batch0 < my_jobs; batch0 += BATCH) {
     const int nb = min(BATCH, my_jobs - batch0);
     for (int jb = 0; jb < nb; ++jb) {
@@ -249,11 +259,14 @@ stream_gemm_kernel(const Params p) {
 #pragma unroll
           for (int ci = 0; ci < (NCH ? NCH : 1); ++ci) consume(acc, bres[ci]);
         } else {
-          uint4 bcur[4], bnext[4];
           float unused = 0.f;
-          load_frag<false>(p, (warp * nchw) * CK, g, t, bcur, unused);
           for (int ci = 0; ci < nchw; ++ci) {
-            if (ci + 1 < nchw) load_frag<false>(p, (warp * nchw + ci + 1) * CK, g, t, bnext, unused);
+            // the next chunk's fragments, one chunk ahead also across tiles and jobs
+            const bool more = ci + 1 < nchw || tile + 1 < TILES || batch0 + jb + 1 < my_jobs;
+            if (more) {
+              const int nj = ci + 1 < nchw || tile + 1 < TILES ? batch0 + jb : batch0 + jb + 1;
+              load_frag<false>(p, (warp * nchw + (ci + 1 < nchw ? ci + 1 : 0)) * CK, g, t, bnext, unused, x_offset(nj));
+            }
             consume(acc, bcur);
 #pragma unroll
             for (int kb = 0; kb < 4; ++kb) bcur[kb] = bnext[kb];
@@ -341,7 +354,7 @@ int launch(const Params& p, int ctas, cudaStream_t s) {
 
 template <int EPI, bool NORM>
 int launch_nch(const Params& p, int ctas, cudaStream_t s) {
-  switch (p.nchw) {
+  switch (p.x_rows ? 0 : p.nchw) {               // operand columns that change from job to job: fragments chunk by chunk
     case 1: return launch<EPI, NORM, 1>(p, ctas, s);
     case 2: return launch<EPI, NORM, 2>(p, ctas, s);
     case 3: return launch<EPI, NORM, 3>(p, ctas, s);
@@ -418,6 +431,17 @@ RLLM_API int rllm_stream_gemm(int epi, const void* X, long long ldx, const float
   p.h = h; p.ldh = ldh; p.rows = rows; p.g = g; p.g_is_bf16 = g_dt == DT_BF16; p.eps = eps;
   p.C = Cout; p.ldc = ldc; p.T = T; p.act = act;
   return run(epi, norm, p, sm_count, (cudaStream_t)stream);
+}
+
+// C[T, N] = one product per group of weight rows, T <= 8: rows n of W in group n / x_rows multiply X's columns from
+// (n / x_rows) * x_gs on (the last group may be shorter). bf16, store epilogue; x_rows and N multiples of 16, x_gs of 8.
+RLLM_API int rllm_stream_gemm_mixes(const void* X, long long ldx, int x_rows, long long x_gs, const void* W, void* Cout,
+                                    long long ldc, int T, int N, int K, int sm_count, void* stream) {
+  if (x_rows <= 0 || x_rows % 16 || x_gs % 8) return ERR_BAD_SIZE;
+  Params p = {};
+  p.W = (const bf16*)W; p.N = N; p.K = K; p.x = (const bf16*)X; p.ldx = ldx; p.x_rows = x_rows; p.x_gs = x_gs;
+  p.C = Cout; p.ldc = ldc; p.T = T;
+  return run(EPI_STORE, false, p, sm_count, (cudaStream_t)stream);
 }
 
 // The q/k/v projection for T <= 8 with the rotation of q and k (pairs d, d + hd/2 of every head, the

@@ -225,7 +225,9 @@ class Backend:
         T, G, K = x.shape
         N = int(rows_each)
         out = torch.empty((T, w.shape[0]), dtype=x.dtype, device=x.device)
-        if self._sm100 is None or T <= 32:
+        if self._sm100 is not None and T <= 8 and self._sm100.gemm_mixes(x, w, N, out):
+            return out
+        if self._sm100 is None or T <= 64:
             return self._mix.grouped_gemm_uniform(x.view(T, G * K), K, w, out, N, self._mix.GEPI_STORE, rows_each=N)
         for g in range(G):
             wg, xg, og = w[g * N: (g + 1) * N], x[:, g], out[:, g * N: g * N + N]

@@ -12,6 +12,7 @@ ranges of keys) were tuned with, and the small case a profiler is pointed at.
     python -m rllm_b200.kernels.microbench gla --heads 16 --dim 128 --vdim 128 --tokens 2048 [--batch 8]
     python -m rllm_b200.kernels.microbench sink --heads 32 --kv-heads 8 --dim 64 --vdim 48 --tokens 2048 --batch 8,64 --context 1024
     python -m rllm_b200.kernels.microbench bounded --heads 16 --kv-heads 4 --dim 128 --vdim 128 --tokens 2048 --batch 8,64
+    python -m rllm_b200.kernels.microbench timemix --heads 16 --dim 128 --width 2048 --tokens 2048 --batch 8,64
     ... --plain 3      # no timing: three plain launches and a synchronize (for ncu -k ... -c ...)
 
 Timing: the kernel runs back to back over `--copies` distinct weight (or cache) tensors, larger
@@ -561,6 +562,67 @@ def cmd_bounded(a) -> None:
     sm100.check_error(DEV)
 
 
+def cmd_timemix(a) -> None:
+    """The kernels of time mixing and of its layers, each beside its like kernel at the same sizes: the scan with a bonus
+    beside gated linear attention's (one kernel, other branches), norm and token shift beside the plain norm, the decays,
+    the products of five mixes beside one product of the same weights, the corrected router beside the plain one, the
+    sum of a layer's terms with and without a gated summand, the values' product with a gate per number."""
+    from . import hybrid, mix
+    H, d, W, rank, E, top = a.heads, a.dim, a.width, a.decay_rank, a.experts, a.top
+    C = H * d
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=DEV)
+    bf = lambda *shape: torch.randn(*shape, device=DEV, dtype=torch.bfloat16)
+    u, mu = torch.randn(H, d, device=DEV), torch.rand(5, W, device=DEV)
+    w1, w2n = torch.ones(W, device=DEV), torch.ones(W, device=DEV)
+    for batch, new in [(1, T) for T in a.tokens] + [(B, 1) for B in a.batch]:
+        T, what = batch * new, f"{batch} x {new}"
+        cu, slots = (torch.arange(batch + 1, dtype=torch.int32) * new).to(DEV), torch.arange(batch, dtype=torch.int32).to(DEV)
+        seq = torch.arange(batch, device=DEV, dtype=torch.int32).repeat_interleave(new).contiguous()
+        proj, alpha = bf(T, 4 * C) * 0.3, torch.rand(T, C, device=DEV) * 0.1 + 0.9
+        states = [torch.zeros(batch, H, d, d, device=DEV) for _ in range(a.copies if new == 1 else 1)]
+        chunk = a.chunk if new >= 3 * a.chunk else 0
+        nb, fl = T * C * (3 * 2 + 8) + 2 * batch * H * d * d * 4, (5.0 if chunk == 0 else 8.0) * T * H * d * d
+        for bonus in (u, None):
+            run([lambda s=s, b=bonus: mix.gla_scan(proj, 0, C, 2 * C, alpha, 1.0, H, d, d, cu, batch, slots, s, chunk, bonus=b)
+                 for s in states] * (1 if new == 1 else 4), a.plain,
+                f"{'scan with bonus' if bonus is not None else '  like: scan of gated linear attention'} {what} tokens, {H} heads of {d}", nb, fl)
+            if a.plain:
+                return
+        h, prev = torch.randn(T, W, device=DEV), torch.zeros(batch, W, device=DEV)
+        run([lambda: mix.shift_mix(h, w1, 1e-6, torch.bfloat16, mu, seq, cu, batch, slots, prev, second=(w2n, 1e-6))] * 4, 0,
+            f"norm, shift and five mixes, second norm {what}", T * W * (4 + 6 * 2))
+        run([lambda: ops.rmsnorm(h, w1, 1e-6, torch.bfloat16)] * 4, 0, f"  like: norm {what}", T * W * 6)
+        z, wz, b0 = bf(T, rank), bf(C, rank), torch.randn(C, device=DEV)
+        run([lambda: mix.lowrank_decay(z, wz, b0)] * 4, 0, f"decays {what}, rank {rank}", C * rank * 2 + T * C * 4, 2.0 * T * C * rank)
+        zf, bb = torch.randn(T, C, device=DEV), torch.randn(C, device=DEV)
+        run([lambda: (sm100.gemm(z, wz, ops.EPI_STORE_F32, out=zf), mix.gla_decay(zf, bb, 16.0))] * 4, 0,
+            f"  like: product and decays of gated linear attention {what}", C * rank * 2 + T * C * 4, 2.0 * T * C * rank)
+        from .backend import Backend
+        be = Backend(torch.bfloat16)
+        x, ws = bf(T, 5, W), [bf(4 * C + rank, W) for _ in range(a.copies)]
+        x0 = x[:, 0].contiguous()
+        run([lambda w=w: be.linear_mixes(x, w, C) for w in ws], 0, f"products of five mixes {what}, {W} -> 4 x {C} + {rank}",
+            (4 * C + rank) * W * 2, 2.0 * T * (4 * C + rank) * W)
+        run([lambda w=w: be.linear(x0, w) for w in ws], 0, f"  like: one product of as many weights {what}",
+            (4 * C + rank) * W * 2, 2.0 * T * (4 * C + rank) * W)
+        del ws
+        z, corr = torch.randn(T, (E + 16) // 16 * 16, device=DEV), torch.randn(E, device=DEV) * 0.1
+        run([lambda: mix.moe_topk(z, top, a.groups, a.keep, True, "sigmoid", experts=E, correction=corr, group_sum=2,
+                                  sum_eps=1e-20, scale=2.5)] * 4, 0, f"corrected router {what}, {E} experts top {top}", z.numel() * 4)
+        ze = z[:, :E].contiguous()
+        run([lambda: mix.moe_topk(ze, top, a.groups, a.keep)] * 4, 0, f"  like: router {what}", ze.numel() * 4)
+        ys, m, s2 = torch.randn(T, top, W, device=DEV), torch.randn(T, W, device=DEV), torch.randn(T, W, device=DEV)
+        for gate in (z[:, E:], None):
+            run([lambda g=gate: hybrid.combine(h, plain=[m, ys, s2], gate=g)] * 4, 0,
+                f"{'sum of terms with a gated one' if gate is not None else '  like: sum of terms'} {what}", (top + 4) * T * W * 4)
+        o, wv, att = bf(T, H * 512), bf(H, 128, 512), torch.empty(T, H * 128, device=DEV, dtype=torch.bfloat16)
+        gf, gh = bf(T, H * 128), bf(T, H)
+        for cols in (True, False):
+            run([lambda c=cols: mix.grouped_gemm_uniform(o, 512, wv, att, 128, mix.GEPI_STORE, gate=gf if c else gh, gate_cols=c)] * 4,
+                0, f"{'values out of latents, a gate per number' if cols else '  like: a gate per head'} {what}",
+                wv.numel() * 2 + T * H * 640 * 2, 2.0 * T * H * 128 * 512)
+
+
 def _delta_pair(hybrid, S, n, W) -> None:
     """S sequences of n tokens, heads of 128 x 128 as wide together as the model."""
     H, d, v, T = max(1, W // 128), 128, 128, S * n
@@ -632,6 +694,14 @@ def main(argv=None) -> int:
     p.add_argument("--softcap", type=float, default=30.0)
     for k, v in (("heads", 16), ("kv-heads", 4), ("dim", 128), ("vdim", 128), ("page", 16), ("context", 1024), ("width", 2048)):
         p.add_argument("--" + k, type=int, default=v)
+    p = sub.add_parser("timemix")
+    p.add_argument("--plain", type=int, default=0, help="N plain launches of the scan instead of timing")
+    p.add_argument("--copies", type=int, default=8)
+    p.add_argument("--tokens", type=ints, default=[2048])
+    p.add_argument("--batch", type=ints, default=[8, 64])
+    for k, v in (("heads", 16), ("dim", 128), ("width", 2048), ("decay-rank", 64), ("chunk", 128), ("experts", 16), ("top", 6),
+                 ("groups", 4), ("keep", 2)):
+        p.add_argument("--" + k, type=int, default=v)
     p = sub.add_parser("talk")
     p.add_argument("--plain", type=int, default=0, help="N plain launches of the prompt kernel instead of timing")
     p.add_argument("--tokens", type=ints, default=[2048])
@@ -684,7 +754,7 @@ def main(argv=None) -> int:
         return 1
     {"gemm": cmd_gemm, "attn-decode": cmd_attn_decode, "attn-prefill": cmd_attn_prefill, "sample": cmd_sample,
      "experts": cmd_experts, "latent-attn": cmd_latent_attn, "gla": cmd_gla, "sink": cmd_sink, "talk": cmd_talk,
-     "scan": cmd_scan, "gated": cmd_gated, "bounded": cmd_bounded}[a.cmd](a)
+     "scan": cmd_scan, "gated": cmd_gated, "bounded": cmd_bounded, "timemix": cmd_timemix}[a.cmd](a)
     return 0
 
 

@@ -23,6 +23,7 @@ ops.register_signatures("sm100", {
     "rllm_stream_gemm_supported": [c_int, c_int, c_int, c_int, c_int, c_int],
     "rllm_stream_gemm": [c_int, _P, c_longlong, _P, c_longlong, _P, _P, c_int, c_float, _P, _P, c_longlong, c_int,
                          c_int, c_int, c_int, _P],
+    "rllm_stream_gemm_mixes": [_P, c_longlong, c_int, c_longlong, _P, _P, c_longlong, c_int, c_int, c_int, c_int, _P],
     "rllm_stream_gemm_qkv_rope": [_P, c_longlong, _P, c_longlong, _P, c_int, c_float, _P, _P, c_longlong, c_int, c_int,
                                   _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, _P],
     "rllm_wait_probe": [_P, c_longlong, c_int, _P],
@@ -168,6 +169,21 @@ def gemm(x: torch.Tensor, w: torch.Tensor, epilogue: int, out: torch.Tensor | No
         int(split), st.err.data_ptr(), st.sm_count, ops._stream())
     ops._check(rc, "tc_gemm")
     return out
+
+
+def gemm_mixes(x: torch.Tensor, w: torch.Tensor, rows_each: int, out: torch.Tensor) -> bool:
+    """out[:, n] = x[:, n // rows_each] w[n]^T for a step of at most 8 tokens on the weight-streaming kernel, one launch;
+    x [T, G, K] contiguous, w [R, K], out [T, R], bfloat16. False (nothing launched) where it does not take the sizes."""
+    T, G, K = x.shape
+    N = w.shape[0]
+    if rows_each % 16 or K % 8 or x.dtype != torch.bfloat16 or not x.is_contiguous() or not stream_supported(ops.EPI_STORE, False, T, N, K) \
+            or x.data_ptr() % 16 or w.data_ptr() % 16 or (N + rows_each - 1) // rows_each > G:
+        return False
+    st = init(x.device)
+    ops._check(ops._fn("sm100", "rllm_stream_gemm_mixes")(
+        x.data_ptr(), x.stride(0), int(rows_each), x.stride(1), w.data_ptr(), out.data_ptr(), out.stride(0), T, N, K, st.sm_count,
+        ops._stream()), "stream_gemm_mixes")
+    return True
 
 
 _norm_max = None

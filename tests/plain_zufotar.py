@@ -221,3 +221,10 @@ def forward(cfg, w, ids, keep_layers=False):
         seen.append(x)
     logits = softcap(rms_norm(x, w["final.norm"], eps) @ w["embed"].T, cfg.get("logit_softcap"))
     return (logits, torch.stack(seen)) if keep_layers else logits
+
+
+def greedy(cfg, w, prompt, n):
+    toks = list(prompt)
+    for _ in range(n):
+        toks.append(int(forward(cfg, w, toks)[-1].argmax()))
+    return toks[len(prompt):]
