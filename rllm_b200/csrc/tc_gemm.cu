@@ -154,6 +154,7 @@ struct Params {
   int splits;         // CTAs per cluster = ranges of K
   int bn;             // persistent kernel: tokens per tile (a multiple of 16, at most the template's BN)
   int* err;           // device error word (0 = fine)
+  int x_rows, x_gs;   // x_rows > 0: weight rows in groups of that many (a multiple of BM), group g reads X's columns from g * x_gs on
   int act;            // store epilogue only: 0 the value as it is, 1 max(value, 0)^2, 2 gelu in its tanh form, 3 gelu in its erf form
   RopeArgs rope;
   NormArgs norm;      // NORM variants only
@@ -307,6 +308,7 @@ tc_gemm_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_constant
     if (lane == 0) {
       const uint64_t pol_w = policy_evict_first();   // weights are read once per step
       const uint64_t pol_x = policy_evict_last();    // the token tile is shared by every weight tile
+      const int x0 = p.x_rows ? n0 / p.x_rows * p.x_gs : 0;
       // weights of the first stages do not depend on the kernel before this one
       const int pre = n_kb < C::STAGES ? n_kb : C::STAGES;
       for (int i = 0; i < pre; ++i) {
@@ -320,7 +322,7 @@ tc_gemm_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_constant
         pdl_wait();                                  // activations come from the kernel before
         for (int i = 0; i < pre; ++i) {
           uint8_t* st = smem + (size_t)i * C::STAGE_BYTES;
-          tma_load_2d_hint(st + W_BYTES, &tmap_x, &full_bar[i], (kb_begin + i) * BK, t0, pol_x);
+          tma_load_2d_hint(st + W_BYTES, &tmap_x, &full_bar[i], x0 + (kb_begin + i) * BK, t0, pol_x);
         }
       }
       int issued = pre;
@@ -333,7 +335,7 @@ tc_gemm_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_constant
         const int k = (kb_begin + i) * BK;
         tma_load_2d_hint(st, &tmap_w, &full_bar[s], k, n0, pol_w);
         if (DUAL) tma_load_2d_hint(st + C::A_BYTES, &tmap_w, &full_bar[s], k, p.up_row0 + n0, pol_w);
-        if (!NORM) tma_load_2d_hint(st + W_BYTES, &tmap_x, &full_bar[s], k, t0, pol_x);
+        if (!NORM) tma_load_2d_hint(st + W_BYTES, &tmap_x, &full_bar[s], x0 + k, t0, pol_x);
         issued = i + 1;
       }
       if (abort_flag) {
@@ -778,6 +780,7 @@ tc_gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmap_w, const __gr
       bool ok = true;
       for (int tile = blockIdx.x; tile < tiles && ok; tile += gridDim.x) {
         const int t0 = (tile % t_tiles) * bn, n0 = (tile / t_tiles) * WR;
+        const int x0 = p.x_rows ? n0 / p.x_rows * p.x_gs : 0;
         for (int kb = 0; kb < n_kb; ++kb, ++it) {
           const int s = it % C::STAGES;
           const uint32_t ph = (uint32_t)(it / C::STAGES) & 1u;
@@ -789,7 +792,7 @@ tc_gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmap_w, const __gr
           const int k = kb * BK;
           tma_load_2d(st, &tmap_w, &full_bar[s], k, n0);
           if (DUAL) tma_load_2d(st + C::A_BYTES, &tmap_w, &full_bar[s], k, p.up_row0 + n0);
-          tma_load_2d_hint(st + C::W_BYTES, &tmap_x, &full_bar[s], k, t0, pol_x);
+          tma_load_2d_hint(st + C::W_BYTES, &tmap_x, &full_bar[s], x0 + k, t0, pol_x);
           issued = it + 1;
         }
       }
@@ -1467,7 +1470,8 @@ void plan(int epi, int T, int N, int K, int sm_count, int allow_split, int* bn_o
 
 // X null: the fused-norm variants (norm must be given, T <= NORM_MAX_T).
 int run(int epi, const void* X, long long ldx, const NormArgs* norm, const void* W, void* Cout, long long ldc,
-        int T, int N, int K, int allow_split, int* err, int sm_count, const RopeArgs* rope, void* stream) {
+        int T, int N, int K, int allow_split, int* err, int sm_count, const RopeArgs* rope, void* stream, int x_rows = 0,
+        int x_gs = 0) {
   if (T <= 0 || N <= 0) return 0;
   if (K <= 0 || K % 8) return ERR_BAD_SIZE;                          // TMA: strides multiple of 16 bytes
   if ((uintptr_t)W & 15) return ERR_BAD_ALIGN;
@@ -1489,13 +1493,14 @@ int run(int epi, const void* X, long long ldx, const NormArgs* norm, const void*
   CUtensorMap mw, mx;
   if ((rc = cached_map(&mw, W, dual ? 2LL * N : N, K, K, BM))) return rc;
   // long portions: a tile of 256 weight rows x bn tokens on a pair of CTAs, each loading half of the token tile
-  const bool pair = g_pairs && !norm && epi != EPI_QKV_ROPE && sm_count >= 2 && many && T >= (dual ? 128 : 256);
+  const bool pair = g_pairs && !norm && !x_rows && epi != EPI_QKV_ROPE && sm_count >= 2 && many && T >= (dual ? 128 : 256);
   if (pair) bn = dual ? 128 : 256;                                   // the pair kernel's tile is fixed
   if (norm) mx = mw;                                                 // not used by the kernel
-  else if ((rc = make_map(&mx, X, T, K, ldx, pair ? bn / 2 : bn))) return rc;
+  else if ((rc = make_map(&mx, X, T, x_rows ? (long long)((N - 1) / x_rows) * x_gs + K : K, ldx, pair ? bn / 2 : bn))) return rc;
   Params p;
   p.C = Cout; p.ldc = (int)ldc; p.T = T; p.N = N; p.K = K; p.up_row0 = N; p.splits = splits; p.err = err; p.bn = bn;
   p.act = epi == EPI_STORE ? t_store_act : 0;
+  p.x_rows = x_rows; p.x_gs = x_gs;
   p.rope = rope ? *rope : RopeArgs{};
   p.norm = norm ? *norm : NormArgs{};
   dim3 grid((T + bn - 1) / bn, (N + BM - 1) / BM, splits);
@@ -1576,6 +1581,15 @@ RLLM_API int rllm_tc_gemm(int epi, const void* X, long long ldx, const void* W, 
   const StoreAct sa(epi);
   if (epi < 0 || epi > 3 || !X) return ERR_BAD_SIZE;
   return run(epi, X, ldx, nullptr, W, Cout, ldc, T, N, K, allow_split, err, sm_count, nullptr, stream);
+}
+
+// One product per group of weight rows, in one launch: rows n of W in group n / x_rows multiply X's columns from
+// (n / x_rows) * x_gs on (the last group may be shorter). Store epilogue; x_rows a multiple of the 128 rows of a tile, K of
+// the 64 values of a stage (a stage never reaches into the next group's columns), x_gs of 8.
+RLLM_API int rllm_tc_gemm_mixes(const void* X, long long ldx, int x_rows, int x_gs, const void* W, void* Cout, long long ldc,
+                                int T, int N, int K, int* err, int sm_count, void* stream) {
+  if (!X || x_rows <= 0 || x_rows % BM || x_gs % 8 || x_gs < K || K % BK) return ERR_BAD_SIZE;
+  return run(EPI_STORE, X, ldx, nullptr, W, Cout, ldc, T, N, K, 1, err, sm_count, nullptr, stream, x_rows, x_gs);
 }
 
 // The same product with RMSNorm in front, in one kernel: X[t, :] = h[row(t), :] * rsqrt(mean(h^2) + eps) * g,

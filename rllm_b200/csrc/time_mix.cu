@@ -8,8 +8,8 @@
 //   A row's norm is the same bits whichever CTA makes it. Without sequences (`token_seq` null) it is two norms of the
 //   same rows in one pass.
 // lowrank_decay: a = exp(-exp(W2 tanh(z) + b)) per column, z a row of `rank` numbers (the first projection's output). A thread
-//   owns columns and walks the rank for eight tokens at a time, whose tanh(z) lie in shared memory; for steps of few
-//   tokens eight lanes share a column and deal the rank out between them.
+//   owns columns and walks the rank for some tokens at a time, whose tanh(z) lie in shared memory; for steps of few
+//   tokens the warps of a CTA deal the rank out between them. W2 is kept transposed, so that a warp reads runs of it.
 #include <initializer_list>
 #include "common.cuh"
 using namespace rllm;
@@ -49,8 +49,10 @@ __device__ __forceinline__ void get(const float* p, float (&v)[VEC]) {
 
 // NV: pieces of VEC numbers a thread has of a row, held in registers (0: any number, the rows are read again). A CTA takes
 // `per` tokens in order; what a token's norm gave serves the next one as the row before.
-template <typename TO, int VEC, int NV>
-__global__ void shift_mix_kernel(const ShiftArgs a, int T, int per) {
+// NMIX: the number of mixes where it is known when compiled; their shares, and the second norm's weight, then also stay
+// in registers (0: any number, read where they are used).
+template <typename TO, int VEC, int NV, int NMIX>
+__global__ void __launch_bounds__(512) shift_mix_kernel(const ShiftArgs a, int T, int per) {
   pdl_launch();
   __shared__ float red[2][32];
   const int W = a.W, step = blockDim.x * VEC, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
@@ -64,12 +66,18 @@ __global__ void shift_mix_kernel(const ShiftArgs a, int T, int per) {
     id = a.state_slots ? a.state_slots[seq] : -1;
   };
   if (a.token_seq) find(t);
-  float w[N][VEC];
+  float w[N][VEC], mus[NMIX ? NMIX : 1][N][VEC], w2[N][VEC];
   if (NV) {
 #pragma unroll
     for (int q = 0; q < N; ++q) {
       const int i = threadIdx.x * VEC + q * step;
-      if (i < W) get<VEC>(a.w + i, w[q]);
+      if (i >= W) continue;
+      get<VEC>(a.w + i, w[q]);
+      if (NMIX) {
+#pragma unroll
+        for (int m = 0; m < NMIX; ++m) get<VEC>(a.mu + (size_t)m * W + i, mus[m][q]);
+        if (a.second) get<VEC>(a.w2 + i, w2[q]);
+      }
     }
   }
   pdl_wait();
@@ -82,12 +90,13 @@ __global__ void shift_mix_kernel(const ShiftArgs a, int T, int per) {
     const float* hr = a.h + (size_t)t * W;
     // a second row is normed here: the one before (the CTA's first token), or the portion's last for its slot
     const float* other = before ? (carried ? nullptr : hr - W) : (slot && row1 - 1 > t ? a.h + (size_t)(row1 - 1) * W : nullptr);
-    float y[N][VEC];
+    float y[N][VEC], held[N][VEC];
     float s0 = 0.f, s1 = 0.f;
     for (int q = 0; NV ? q < N : threadIdx.x * VEC + q * step < W; ++q) {
       const int i = threadIdx.x * VEC + q * step, r = NV ? q : 0;
       if (i >= W) break;
       get<VEC>(hr + i, x[r]);
+      if (NV && slot) get<VEC>(slot + i, held[r]);
 #pragma unroll
       for (int e = 0; e < VEC; ++e) s0 = fmaf(x[r][e], x[r][e], s0);
       if (other) {
@@ -124,22 +133,35 @@ __global__ void shift_mix_kernel(const ShiftArgs a, int T, int per) {
 #pragma unroll
         for (int e = 0; e < VEC; ++e) p[e] = other ? y[k][e] : o[k][e];
       } else if (slot) {
-        get<VEC>(slot + i, p);
+        if (NV) {
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) p[e] = held[k][e];
+        } else {
+          get<VEC>(slot + i, p);
+        }
         put<float, VEC>(slot + i, other ? y[k] : n);
       }
-      for (int m = 0; m < a.nmix; ++m) {
-        float mu[VEC];
-        get<VEC>(a.mu + (size_t)m * W + i, mu);
+      if (NMIX) {
 #pragma unroll
-        for (int e = 0; e < VEC; ++e) z[e] = fmaf(p[e] - n[e], mu[e], n[e]);
-        put<TO, VEC>((TO*)a.mixes + ((size_t)t * a.nmix + m) * W + i, z);
+        for (int m = 0; m < NMIX; ++m) {
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) z[e] = fmaf(p[e] - n[e], mus[m][k][e], n[e]);
+          put<TO, VEC>((TO*)a.mixes + ((size_t)t * NMIX + m) * W + i, z);
+        }
+      } else {
+        for (int m = 0; m < a.nmix; ++m) {
+          float mu[VEC];
+          get<VEC>(a.mu + (size_t)m * W + i, mu);
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) z[e] = fmaf(p[e] - n[e], mu[e], n[e]);
+          put<TO, VEC>((TO*)a.mixes + ((size_t)t * a.nmix + m) * W + i, z);
+        }
       }
       if (a.plain) put<TO, VEC>((TO*)a.plain + (size_t)t * W + i, n);
       if (a.second) {
-        float w2[VEC];
-        get<VEC>(a.w2 + i, w2);
+        if (!NMIX) get<VEC>(a.w2 + i, w2[k]);
 #pragma unroll
-        for (int e = 0; e < VEC; ++e) z[e] = x[k][e] * r2 * w2[e];
+        for (int e = 0; e < VEC; ++e) z[e] = x[k][e] * r2 * w2[k][e];
         put<TO, VEC>((TO*)a.second + (size_t)t * W + i, z);
       }
       if (NV) {
@@ -153,114 +175,140 @@ __global__ void shift_mix_kernel(const ShiftArgs a, int T, int per) {
 
 constexpr int DT_TOKENS = 8, DT_MAX_RANK = 1024;
 
-// eight numbers of a row of W2
-template <typename TI>
-__device__ __forceinline__ void get8(const TI* p, float (&w)[8]) {
-  if constexpr (sizeof(TI) == 2) {
-    const uint4 u = *reinterpret_cast<const uint4*>(p);
-    const __nv_bfloat162* h2 = reinterpret_cast<const __nv_bfloat162*>(&u);
-#pragma unroll
-    for (int e = 0; e < 4; ++e) { const float2 f = __bfloat1622float2(h2[e]); w[2 * e] = f.x; w[2 * e + 1] = f.y; }
+// CPT neighbouring numbers of a row of W2^T
+template <typename TI, int CPT>
+__device__ __forceinline__ void get_cols(const TI* p, float (&w)[CPT]) {
+  if constexpr (CPT == 4 && sizeof(TI) == 2) {
+    const uint2 u = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x));
+    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+    w[0] = a.x; w[1] = a.y; w[2] = b.x; w[3] = b.y;
+  } else if constexpr (CPT == 4) {
+    const float4 u = *reinterpret_cast<const float4*>(p);
+    w[0] = u.x; w[1] = u.y; w[2] = u.z; w[3] = u.w;
   } else {
-    const float4 u = *reinterpret_cast<const float4*>(p), v = *reinterpret_cast<const float4*>(p + 4);
-    w[0] = u.x; w[1] = u.y; w[2] = u.z; w[3] = u.w; w[4] = v.x; w[5] = v.y; w[6] = v.z; w[7] = v.w;
+#pragma unroll
+    for (int q = 0; q < CPT; ++q) w[q] = to_f32(p[q]);
   }
 }
-__device__ __forceinline__ void fma8(float w, const float* th, float (&acc)[DT_TOKENS]) {
-  const float4 a = *reinterpret_cast<const float4*>(th), b = *reinterpret_cast<const float4*>(th + 4);
-  acc[0] = fmaf(w, a.x, acc[0]); acc[1] = fmaf(w, a.y, acc[1]); acc[2] = fmaf(w, a.z, acc[2]); acc[3] = fmaf(w, a.w, acc[3]);
-  acc[4] = fmaf(w, b.x, acc[4]); acc[5] = fmaf(w, b.y, acc[5]); acc[6] = fmaf(w, b.z, acc[6]); acc[7] = fmaf(w, b.w, acc[7]);
+template <int N>
+__device__ __forceinline__ void get_tokens(const float* th, float (&v)[N]) {
+#pragma unroll
+  for (int i = 0; i < N; i += 4) {
+    const float4 a = *reinterpret_cast<const float4*>(th + i);
+    v[i] = a.x; v[i + 1] = a.y; v[i + 2] = a.z; v[i + 3] = a.w;
+  }
+}
+// tanh of a tile's rows, [rank][TT] in shared memory (zeros for the rows beyond n)
+template <typename TI, int TT>
+__device__ __forceinline__ void stage_tanh(float* th, const TI* z, long long ld, int rank, int n) {
+  for (int x = threadIdx.x; x < rank * TT; x += blockDim.x) {
+    const int j = x % rank, tt = x / rank;
+    th[j * TT + tt] = tt < n ? tanhf(to_f32(z[tt * ld + j])) : 0.f;
+  }
 }
 
-// Long portions, and sizes the other kernel does not take: CPT columns a thread (blockDim.x apart), the whole rank. VEC: W2's
-// rows are read eight numbers at a time (rank a multiple of 8, rows on 16-byte boundaries).
-template <typename TI, bool VEC, int CPT>
-__global__ void lowrank_decay_kernel(const TI* __restrict__ z, long long ld, int rank, const TI* __restrict__ w2,
-                                     const float* __restrict__ bias, float* __restrict__ out, int T, int C) {
+// Long portions: a thread owns CPT neighbouring columns and walks the whole rank for TT tokens.
+template <typename TI, int CPT, int TT>
+__global__ void __launch_bounds__(128)
+lowrank_decay_kernel(const TI* __restrict__ z, long long ld, int rank, const TI* __restrict__ w2t,
+                     const float* __restrict__ bias, float* __restrict__ out, int T, int C) {
   pdl_launch();
   pdl_wait();
-  extern __shared__ __align__(16) float th[];         // [rank][DT_TOKENS]
-  const int t0 = blockIdx.y * DT_TOKENS, n = min(DT_TOKENS, T - t0);
-  for (int x = threadIdx.x; x < rank * DT_TOKENS; x += blockDim.x) {
-    const int j = x % rank, tt = x / rank;
-    th[j * DT_TOKENS + tt] = tt < n ? tanhf(to_f32(z[(long long)(t0 + tt) * ld + j])) : 0.f;
-  }
+  extern __shared__ __align__(16) float th[];         // [rank][TT]
+  const int t0 = blockIdx.y * TT, n = min(TT, T - t0);
+  stage_tanh<TI, TT>(th, z + (long long)t0 * ld, ld, rank, n);
   __syncthreads();
-  const int c0 = blockIdx.x * blockDim.x * CPT + threadIdx.x;
-  float acc[CPT][DT_TOKENS];
+  const int c = (blockIdx.x * blockDim.x + threadIdx.x) * CPT;       // C is a multiple of CPT
+  if (c >= C) return;
+  float acc[CPT][TT];
 #pragma unroll
   for (int q = 0; q < CPT; ++q)
 #pragma unroll
-    for (int i = 0; i < DT_TOKENS; ++i) acc[q][i] = 0.f;
-  const TI* wr[CPT];                                  // columns beyond C read the last one's row and store nothing
+    for (int i = 0; i < TT; ++i) acc[q][i] = 0.f;
+  const TI* wp = w2t + c;
+#pragma unroll 4
+  for (int j = 0; j < rank; ++j) {
+    float w[CPT], v[TT];
+    get_cols<TI, CPT>(wp + (size_t)j * C, w);
+    get_tokens<TT>(th + j * TT, v);
 #pragma unroll
-  for (int q = 0; q < CPT; ++q) wr[q] = w2 + (size_t)min(c0 + q * (int)blockDim.x, C - 1) * rank;
-  if (VEC) {
-    for (int j = 0; j < rank; j += 8) {
-      float w[CPT][8];
+    for (int q = 0; q < CPT; ++q)
 #pragma unroll
-      for (int q = 0; q < CPT; ++q) get8(wr[q] + j, w[q]);
-#pragma unroll
-      for (int e = 0; e < 8; ++e)
-#pragma unroll
-        for (int q = 0; q < CPT; ++q) fma8(w[q][e], th + (j + e) * DT_TOKENS, acc[q]);
-    }
-  } else {
-    for (int j = 0; j < rank; ++j)
-#pragma unroll
-      for (int q = 0; q < CPT; ++q) fma8(to_f32(wr[q][j]), th + j * DT_TOKENS, acc[q]);
+      for (int i = 0; i < TT; ++i) acc[q][i] = fmaf(w[q], v[i], acc[q][i]);
   }
+  float b[CPT];
 #pragma unroll
-  for (int q = 0; q < CPT; ++q) {
-    const int c = c0 + q * (int)blockDim.x;
-    if (c >= C) continue;
-    const float b = bias[c];
+  for (int q = 0; q < CPT; ++q) b[q] = bias[c + q];
 #pragma unroll
-    for (int i = 0; i < DT_TOKENS; ++i)
-      if (i < n) out[(long long)(t0 + i) * C + c] = expf(-expf(acc[q][i] + b));
+  for (int i = 0; i < TT; ++i) {
+    if (i >= n) break;
+    float* o = out + (long long)(t0 + i) * C + c;
+    float e[CPT];
+#pragma unroll
+    for (int q = 0; q < CPT; ++q) e[q] = expf(-expf(acc[q][i] + b[q]));
+    if constexpr (CPT == 4) *reinterpret_cast<float4*>(o) = make_float4(e[0], e[1], e[2], e[3]);
+    else
+#pragma unroll
+      for (int q = 0; q < CPT; ++q) o[q] = e[q];
   }
 }
 
-// Steps of few tokens: eight neighbouring lanes share a column and eight numbers of every 64 of the rank each; their
-// sums are joined by shuffles in lane order, after which each lane has one token's. The rows of W2, which no kernel
-// writes, are asked for before the wait (the first 64 of the rank). The order of a sum depends on the rank alone.
-template <typename TI>
+// Steps of few tokens: a CTA has 32 * CPT columns and eight tokens; its eight warps take every eighth number of the
+// rank, and their sums meet in shared memory in warp order. A warp's first numbers of W2, which no kernel writes, are
+// asked for before the wait. The order of a sum depends on the rank alone.
+constexpr int DT_AHEAD = 8;
+template <typename TI, int CPT>
 __global__ void __launch_bounds__(256)
-lowrank_decay_few_kernel(const TI* __restrict__ z, long long ld, int rank, const TI* __restrict__ w2,
+lowrank_decay_few_kernel(const TI* __restrict__ z, long long ld, int rank, const TI* __restrict__ w2t,
                          const float* __restrict__ bias, float* __restrict__ out, int T, int C) {
   pdl_launch();
-  extern __shared__ __align__(16) float th[];         // [rank][DT_TOKENS + 4]: lanes eight rows apart meet other banks
-  constexpr int LD = DT_TOKENS + 4;
-  const int part = threadIdx.x & 7, c = blockIdx.x * 32 + (threadIdx.x >> 3), cc = min(c, C - 1);
-  const TI* wr = w2 + (size_t)cc * rank;
-  float w[8];
-  if (part * 8 < rank) get8(wr + part * 8, w);
-  const float b = bias[cc];
+  constexpr int TT = DT_TOKENS, COLS = 32 * CPT;
+  extern __shared__ __align__(16) float th[];         // [rank][TT], then the sums [8][TT][COLS]
+  float* sums = th + rank * TT;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int c = (blockIdx.x * 32 + lane) * CPT, cc = min(c, C - CPT);  // C is a multiple of CPT
+  const TI* wp = w2t + cc;
+  float w[DT_AHEAD][CPT];
+#pragma unroll
+  for (int k = 0; k < DT_AHEAD; ++k)
+    if (warp + 8 * k < rank) get_cols<TI, CPT>(wp + (size_t)(warp + 8 * k) * C, w[k]);
   pdl_wait();
-  const int t0 = blockIdx.y * DT_TOKENS, n = min(DT_TOKENS, T - t0);
-  for (int x = threadIdx.x; x < rank * DT_TOKENS; x += blockDim.x) {
-    const int j = x % rank, tt = x / rank;
-    th[j * LD + tt] = tt < n ? tanhf(to_f32(z[(long long)(t0 + tt) * ld + j])) : 0.f;
-  }
+  const int t0 = blockIdx.y * TT, n = min(TT, T - t0);
+  stage_tanh<TI, TT>(th, z + (long long)t0 * ld, ld, rank, n);
   __syncthreads();
-  float acc[DT_TOKENS];
+  float acc[CPT][TT];
 #pragma unroll
-  for (int i = 0; i < DT_TOKENS; ++i) acc[i] = 0.f;
-  for (int j = part * 8; j < rank; j += 64) {
-    if (j >= 64) get8(wr + j, w);
+  for (int q = 0; q < CPT; ++q)
 #pragma unroll
-    for (int e = 0; e < 8; ++e) fma8(w[e], th + (j + e) * LD, acc);
+    for (int i = 0; i < TT; ++i) acc[q][i] = 0.f;
+  auto add = [&](int j, const float (&wj)[CPT]) {
+    float v[TT];
+    get_tokens<TT>(th + j * TT, v);
+#pragma unroll
+    for (int q = 0; q < CPT; ++q)
+#pragma unroll
+      for (int i = 0; i < TT; ++i) acc[q][i] = fmaf(wj[q], v[i], acc[q][i]);
+  };
+#pragma unroll
+  for (int k = 0; k < DT_AHEAD; ++k)
+    if (warp + 8 * k < rank) add(warp + 8 * k, w[k]);
+  for (int j = warp + 8 * DT_AHEAD; j < rank; j += 8) {
+    get_cols<TI, CPT>(wp + (size_t)j * C, w[0]);
+    add(j, w[0]);
   }
 #pragma unroll
-  for (int i = 0; i < DT_TOKENS; ++i) {
-    acc[i] += __shfl_xor_sync(0xffffffffu, acc[i], 1);
-    acc[i] += __shfl_xor_sync(0xffffffffu, acc[i], 2);
-    acc[i] += __shfl_xor_sync(0xffffffffu, acc[i], 4);
-  }
-  float v = acc[0];
+  for (int q = 0; q < CPT; ++q)
 #pragma unroll
-  for (int i = 1; i < DT_TOKENS; ++i) v = part == i ? acc[i] : v;
-  if (c < C && part < n) out[(long long)(t0 + part) * C + c] = expf(-expf(v + b));
+    for (int i = 0; i < TT; ++i) sums[(warp * TT + i) * COLS + lane + 32 * q] = acc[q][i];
+  __syncthreads();
+  for (int x = threadIdx.x; x < TT * COLS; x += 256) {
+    const int i = x / COLS, s = x % COLS, col = (blockIdx.x * 32 + (s & 31)) * CPT + (s >> 5);
+    float v = 0.f;
+#pragma unroll
+    for (int k = 0; k < 8; ++k) v += sums[(k * TT + i) * COLS + s];
+    if (i < n && col < C) out[(long long)(t0 + i) * C + col] = expf(-expf(v + bias[col]));
+  }
 }
 
 template <typename TO>
@@ -268,15 +316,16 @@ int launch_shift(const ShiftArgs& a, int T, bool vec, cudaStream_t s) {
   const int pieces = a.W / (vec ? 4 : 1);
   const int threads = pieces >= 1024 && vec ? 512 : pieces >= 256 ? 256 : pieces >= 128 ? 128 : 64;
   const int nv = (pieces + threads - 1) / threads;
-  // long portions: four tokens a CTA share the norms of their rows and the shares (mu) in the L1 cache
-  const int per = T >= 1024 ? 4 : 1;
+  // long portions: two tokens a CTA, which share the norms of their rows and the shares of the mixes
+  const int per = T >= 1024 ? 2 : 1;
   const dim3 grid((T + per - 1) / per), block(threads);
-#define GO(V, NV) return launch_ex(shift_mix_kernel<TO, V, NV>, grid, block, 0, s, 1, a, T, per)
-  if (!vec) GO(1, 0);
-  if (nv == 1) GO(4, 1);
-  if (nv == 2) GO(4, 2);
-  if (nv <= 4) GO(4, 4);
-  GO(4, 0);
+#define GO(V, NV, M) return launch_ex(shift_mix_kernel<TO, V, NV, M>, grid, block, 0, s, 1, a, T, per)
+  if (!vec) GO(1, 0, 0);
+  if (nv == 1 && a.nmix == 5) GO(4, 1, 5);
+  if (nv == 2 && a.nmix == 5) GO(4, 2, 5);
+  if (nv <= 2) GO(4, 2, 0);
+  if (nv <= 4) GO(4, 4, 0);
+  GO(4, 0, 0);
 #undef GO
 }
 
@@ -300,30 +349,33 @@ RLLM_API int rllm_shift_mix(int dt, const float* h, const float* w, float eps, c
   return ERR_BAD_DTYPE;
 }
 
-// z: [T, >= rank] of type dt with row stride ld; w2 [C, rank] of type dt; bias float [C]; out float [T, C].
-RLLM_API int rllm_lowrank_decay(int dt, const void* z, long long ld, int rank, const void* w2, const float* bias, float* out,
+// z: [T, >= rank] of type dt with row stride ld; w2t [rank, C] of type dt; bias float [C]; out float [T, C].
+RLLM_API int rllm_lowrank_decay(int dt, const void* z, long long ld, int rank, const void* w2t, const float* bias, float* out,
                                 int T, int C, void* stream) {
   if (T <= 0 || C <= 0) return 0;
   if (rank <= 0 || rank > DT_MAX_RANK) return ERR_BAD_SIZE;
-  const int row_tiles = (T + DT_TOKENS - 1) / DT_TOKENS;
-  if (row_tiles > 65535) return ERR_TOO_LARGE;
-  const bool vec = rank % 8 == 0 && !((uintptr_t)w2 & 15);
+  if (dt != DT_F32 && dt != DT_BF16) return ERR_BAD_DTYPE;
+  if ((T + DT_TOKENS - 1) / DT_TOKENS > 65535) return ERR_TOO_LARGE;
   cudaStream_t s = (cudaStream_t)stream;
-  if (vec && row_tiles < 16) {
-    const dim3 grid((C + 31) / 32, row_tiles);
-    const size_t smem = (size_t)rank * (DT_TOKENS + 4) * sizeof(float);       // at most 48 KB
-    if (dt == DT_F32)
-      return launch_ex(lowrank_decay_few_kernel<float>, grid, dim3(256), smem, s, 1, (const float*)z, ld, rank, (const float*)w2, bias, out, T, C);
-    if (dt == DT_BF16)
-      return launch_ex(lowrank_decay_few_kernel<bf16>, grid, dim3(256), smem, s, 1, (const bf16*)z, ld, rank, (const bf16*)w2, bias, out, T, C);
-    return ERR_BAD_DTYPE;
-  }
-  const int cpt = vec && C >= 512 ? 4 : 1;
-  const dim3 grid((C + 128 * cpt - 1) / (128 * cpt), row_tiles);
-  const size_t smem = (size_t)rank * DT_TOKENS * sizeof(float);
-#define GO(TI, V, N) return launch_ex(lowrank_decay_kernel<TI, V, N>, grid, dim3(128), smem, s, 1, (const TI*)z, ld, rank, (const TI*)w2, bias, out, T, C)
-  if (dt == DT_F32) { if (cpt == 4) GO(float, true, 4); if (vec) GO(float, true, 1); GO(float, false, 1); }
-  if (dt == DT_BF16) { if (cpt == 4) GO(bf16, true, 4); if (vec) GO(bf16, true, 1); GO(bf16, false, 1); }
+  const bool four = C % 4 == 0 && !((uintptr_t)w2t & 15) && !((uintptr_t)out & 15);
+  if (T <= 16 * DT_TOKENS) {
+    const int cpt = C % 2 == 0 ? 2 : 1;
+    const dim3 grid((C + 32 * cpt - 1) / (32 * cpt), (T + DT_TOKENS - 1) / DT_TOKENS);
+    const size_t smem = ((size_t)rank * DT_TOKENS + 8 * DT_TOKENS * 32 * cpt) * sizeof(float);      // at most 48 KB
+#define GO(TI, N) return launch_ex(lowrank_decay_few_kernel<TI, N>, grid, dim3(256), smem, s, 1, (const TI*)z, ld, rank, (const TI*)w2t, bias, out, T, C)
+    if (dt == DT_F32) { if (cpt == 2) GO(float, 2); GO(float, 1); }
+    if (cpt == 2) GO(bf16, 2);
+    GO(bf16, 1);
 #undef GO
-  return ERR_BAD_DTYPE;
+  }
+  // tokens a tile: 16 where their shared memory and registers leave room
+  const int cpt = four ? 4 : 1, tt = four && rank <= 512 ? 16 : 8;
+  const dim3 grid((C + 128 * cpt - 1) / (128 * cpt), (T + tt - 1) / tt);
+  const size_t smem = (size_t)rank * tt * sizeof(float);                                             // at most 32 KB
+#define GO(TI, N, TT) return launch_ex(lowrank_decay_kernel<TI, N, TT>, grid, dim3(128), smem, s, 1, (const TI*)z, ld, rank, (const TI*)w2t, bias, out, T, C)
+  if (dt == DT_F32) { if (tt == 16) GO(float, 4, 16); if (four) GO(float, 4, 8); GO(float, 1, 8); }
+  if (tt == 16) GO(bf16, 4, 16);
+  if (four) GO(bf16, 4, 8);
+  GO(bf16, 1, 8);
+#undef GO
 }

@@ -220,12 +220,13 @@ class Backend:
 
     def linear_mixes(self, x, w, rows_each, tag=None):
         """One product per mix of the input, side by side: out[:, g*N + n] = x[:, g] w[g*N + n]^T with N = rows_each, in the
-        run dtype; x [T, G, K], w [R, K] the problems' rows under each other, the last one with what is left of R. Steps
-        of few tokens run as one launch that streams all weights, longer ones as a tensor-core product each."""
+        run dtype; x [T, G, K], w [R, K] the problems' rows under each other, the last one with what is left of R. One
+        launch, on the weight-streaming or the tcgen05 kernel where they take the sizes (weight tiles that do not straddle two
+        problems), else on the grouped product; long portions whose sizes only the plain product takes: one each."""
         T, G, K = x.shape
         N = int(rows_each)
         out = torch.empty((T, w.shape[0]), dtype=x.dtype, device=x.device)
-        if self._sm100 is not None and T <= 8 and self._sm100.gemm_mixes(x, w, N, out):
+        if self._sm100 is not None and self._sm100.gemm_mixes(x, w, N, out):
             return out
         if self._sm100 is None or T <= 64:
             return self._mix.grouped_gemm_uniform(x.view(T, G * K), K, w, out, N, self._mix.GEPI_STORE, rows_each=N)
@@ -431,8 +432,8 @@ class Backend:
                                            prev, second=second)
         return mixes, n2
 
-    def lowrank_decay(self, z, w2, bias):
-        return self._mix.lowrank_decay(z, w2, bias)
+    def lowrank_decay(self, z, w2_t, bias):
+        return self._mix.lowrank_decay(z, w2_t, bias)
 
     # ---- recurrent mixers with a short convolution, attention with mixed heads, layers whose sublayers run side by
     # side (libraries "recurrent", "rows" and "hybrid")

@@ -593,7 +593,8 @@ def cmd_timemix(a) -> None:
             f"norm, shift and five mixes, second norm {what}", T * W * (4 + 6 * 2))
         run([lambda: ops.rmsnorm(h, w1, 1e-6, torch.bfloat16)] * 4, 0, f"  like: norm {what}", T * W * 6)
         z, wz, b0 = bf(T, rank), bf(C, rank), torch.randn(C, device=DEV)
-        run([lambda: mix.lowrank_decay(z, wz, b0)] * 4, 0, f"decays {what}, rank {rank}", C * rank * 2 + T * C * 4, 2.0 * T * C * rank)
+        wt = wz.t().contiguous()
+        run([lambda: mix.lowrank_decay(z, wt, b0)] * 4, 0, f"decays {what}, rank {rank}", C * rank * 2 + T * C * 4, 2.0 * T * C * rank)
         zf, bb = torch.randn(T, C, device=DEV), torch.randn(C, device=DEV)
         run([lambda: (sm100.gemm(z, wz, ops.EPI_STORE_F32, out=zf), mix.gla_decay(zf, bb, 16.0))] * 4, 0,
             f"  like: product and decays of gated linear attention {what}", C * rank * 2 + T * C * 4, 2.0 * T * C * rank)

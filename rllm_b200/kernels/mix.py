@@ -446,15 +446,15 @@ def shift_mix(h: torch.Tensor, w: torch.Tensor, eps: float, out_dtype: torch.dty
     return mixes, out, out2
 
 
-def lowrank_decay(z: torch.Tensor, w2: torch.Tensor, bias: torch.Tensor) -> torch.Tensor:
-    """float32 [T, C]: exp(-exp(w2 tanh(z) + bias)); z [T, rank] (unit inner stride) and w2 [C, rank] of one dtype."""
-    C, rank = w2.shape
+def lowrank_decay(z: torch.Tensor, w2_t: torch.Tensor, bias: torch.Tensor) -> torch.Tensor:
+    """float32 [T, C]: exp(-exp(W2 tanh(z) + bias)); z [T, rank] (unit inner stride) and w2_t = W2^T [rank, C] of one dtype."""
+    rank, C = w2_t.shape
     _rows(z, "z", rank)
-    _cuda(w2, "w2")
-    if z.dtype != w2.dtype or not w2.is_contiguous() or z.shape[1] != rank:
-        raise KernelError(f"lowrank_decay: z must be [T, {rank}] of w2's dtype, w2 contiguous")
+    _cuda(w2_t, "w2_t")
+    if z.dtype != w2_t.dtype or not w2_t.is_contiguous() or z.shape[1] != rank:
+        raise KernelError(f"lowrank_decay: z must be [T, {rank}] of w2_t's dtype, w2_t contiguous")
     _f32(bias, "decay bias", (C,))
     out = torch.empty((z.shape[0], C), dtype=torch.float32, device=z.device)
-    _check(_fn("mix", "rllm_lowrank_decay")(_dt(z, "z"), z.data_ptr(), z.stride(0), rank, w2.data_ptr(), bias.data_ptr(),
+    _check(_fn("mix", "rllm_lowrank_decay")(_dt(z, "z"), z.data_ptr(), z.stride(0), rank, w2_t.data_ptr(), bias.data_ptr(),
                                             out.data_ptr(), z.shape[0], C, _stream()), "lowrank_decay")
     return out

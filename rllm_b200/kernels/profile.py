@@ -165,10 +165,10 @@ class OpProfile:
     def norm_pair(self, h, *a):
         return self._timed("norm", h.numel() * (4 + 2 * self._be.dtype.itemsize), 0, self._be.norm_pair, h, *a)
 
-    def lowrank_decay(self, z, w2, bias):
-        T, (C, rank) = z.shape[0], w2.shape
-        return self._timed("decay", _nbytes(w2) + T * (rank * z.element_size() + 4 * C), 2 * T * C * rank, self._be.lowrank_decay,
-                           z, w2, bias)
+    def lowrank_decay(self, z, w2_t, bias):
+        T, (rank, C) = z.shape[0], w2_t.shape
+        return self._timed("decay", _nbytes(w2_t) + T * (rank * z.element_size() + 4 * C), 2 * T * C * rank, self._be.lowrank_decay,
+                           z, w2_t, bias)
 
     def softcap(self, x, cap):
         return self._timed("softcap", 2 * _nbytes(x), 0, self._be.softcap, x, cap)

@@ -12,6 +12,7 @@ from . import ops
 _P = c_void_p
 ops.register_signatures("sm100", {
     "rllm_tc_gemm": [c_int, _P, c_longlong, _P, _P, c_longlong, c_int, c_int, c_int, c_int, _P, c_int, _P],
+    "rllm_tc_gemm_mixes": [_P, c_longlong, c_int, c_int, _P, _P, c_longlong, c_int, c_int, c_int, _P, c_int, _P],
     "rllm_tc_gemm_set_pairs": [c_int],
     "rllm_tc_gemm_set_token_rows": [c_int],
     "rllm_tc_gemm_plan": [c_int, c_int, c_int, c_int, c_int, c_int, POINTER(c_int), POINTER(c_int)],
@@ -172,14 +173,22 @@ def gemm(x: torch.Tensor, w: torch.Tensor, epilogue: int, out: torch.Tensor | No
 
 
 def gemm_mixes(x: torch.Tensor, w: torch.Tensor, rows_each: int, out: torch.Tensor) -> bool:
-    """out[:, n] = x[:, n // rows_each] w[n]^T for a step of at most 8 tokens on the weight-streaming kernel, one launch;
-    x [T, G, K] contiguous, w [R, K], out [T, R], bfloat16. False (nothing launched) where it does not take the sizes."""
+    """out[:, n] = x[:, n // rows_each] w[n]^T in one launch: steps of at most 8 tokens on the weight-streaming kernel, longer
+    ones on tcgen05; x [T, G, K] contiguous, w [R, K], out [T, R], bfloat16. False (nothing launched) where neither takes
+    the sizes."""
     T, G, K = x.shape
     N = w.shape[0]
-    if rows_each % 16 or K % 8 or x.dtype != torch.bfloat16 or not x.is_contiguous() or not stream_supported(ops.EPI_STORE, False, T, N, K) \
-            or x.data_ptr() % 16 or w.data_ptr() % 16 or (N + rows_each - 1) // rows_each > G:
+    if K % 8 or x.dtype != torch.bfloat16 or not x.is_contiguous() or x.data_ptr() % 16 or w.data_ptr() % 16 \
+            or (N + rows_each - 1) // rows_each > G:
         return False
     st = init(x.device)
+    if rows_each % 128 == 0 and K % 64 == 0 and N % 4 == 0 and T > 8:
+        ops._check(ops._fn("sm100", "rllm_tc_gemm_mixes")(
+            x.data_ptr(), x.stride(0), int(rows_each), x.stride(1), w.data_ptr(), out.data_ptr(), out.stride(0), T, N, K,
+            st.err.data_ptr(), st.sm_count, ops._stream()), "tc_gemm_mixes")
+        return True
+    if rows_each % 16 or not stream_supported(ops.EPI_STORE, False, T, N, K):
+        return False
     ops._check(ops._fn("sm100", "rllm_stream_gemm_mixes")(
         x.data_ptr(), x.stride(0), int(rows_each), x.stride(1), w.data_ptr(), out.data_ptr(), out.stride(0), T, N, K, st.sm_count,
         ops._stream()), "stream_gemm_mixes")

@@ -108,6 +108,7 @@ class TimeMixing(Part):
         f32 = lambda t: t.float().contiguous()
         self._mu, self._w0, self._u, self._norm_f32 = f32(self.mu).view(5, self.hidden), f32(self.b_w0), f32(self.u), f32(self.w_norm)
         self._rank = self.w_in.shape[0] - 4 * C
+        self._w2_t = self.w_w2.t().contiguous()          # the kernel's lanes own columns
         if self.w_w2.shape[1] != self._rank:
             raise ValueError(f"{self.prefix}w1 has {self._rank} rows, w2 takes {self.w_w2.shape[1]}")
 
@@ -117,7 +118,7 @@ class TimeMixing(Part):
         H, d, C = self.heads, self.dim, self.heads * self.dim
         x, n2 = be.shift_mix(h, norm.weight_f32(), norm.eps, self._mu, ctx, cache.state["prev"], second)    # [T, 5, W]
         proj = be.linear_mixes(x, self.w_in, C, tag="in")                # [T, r | k | v | g | w1]
-        decay = be.lowrank_decay(proj[:, 4 * C:], self.w_w2, self._w0)   # float [T, C]
+        decay = be.lowrank_decay(proj[:, 4 * C:], self._w2_t, self._w0)   # float [T, C]
         o = be.gla_scan(proj, 0, C, 2 * C, decay, 1.0, H, d, d, ctx.cu_q, ctx.num_seqs, ctx.state_slots, cache.state["S"],
                         scan_chunk(ctx, self.chunk), bonus=self._u)
         return be.linear_f32(be.gla_finish(o, self._norm_f32, self.eps, proj, 3 * C), self.w_o, tag="o"), n2
