@@ -48,15 +48,17 @@ __device__ __forceinline__ void get(const float* p, float (&v)[VEC]) {
 }
 
 // NV: pieces of VEC numbers a thread has of a row, held in registers (0: any number, the rows are read again). A CTA takes
-// `per` tokens in order; what a token's norm gave serves the next one as the row before.
+// `per` tokens in order, the next one's row asked for before this one's sum; what a token's norm gave serves the next one
+// as the row before.
 // NMIX: the number of mixes where it is known when compiled; their shares, and the second norm's weight, then also stay
-// in registers (0: any number, read where they are used).
-template <typename TO, int VEC, int NV, int NMIX>
-__global__ void __launch_bounds__(512) shift_mix_kernel(const ShiftArgs a, int T, int per) {
+// in registers (0: any number, read where they are used). SHIFT false: no sequences, every row by itself.
+template <typename TO, int VEC, int NV, int NMIX, bool SHIFT>
+__global__ void __launch_bounds__(512, NV == 1 ? 2 : 1) shift_mix_kernel(const ShiftArgs a, int T, int per) {
   pdl_launch();
   __shared__ float red[2][32];
   const int W = a.W, step = blockDim.x * VEC, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
   constexpr int N = NV ? NV : 1;
+  constexpr bool KEPT = NV && (NMIX || !SHIFT);     // the second norm's weight stays in registers
   // the step's metadata and the norm's weight are written by no kernel of the step: read before the wait
   int t = blockIdx.x * per;
   const int t_end = min(T, t + per);
@@ -65,7 +67,8 @@ __global__ void __launch_bounds__(512) shift_mix_kernel(const ShiftArgs a, int T
     seq = a.token_seq[at]; row0 = a.cu_q[seq]; row1 = a.cu_q[seq + 1];
     id = a.state_slots ? a.state_slots[seq] : -1;
   };
-  if (a.token_seq) find(t);
+  const bool shift = SHIFT && a.token_seq != nullptr;
+  if (shift) find(t);
   float w[N][VEC], mus[NMIX ? NMIX : 1][N][VEC], w2[N][VEC];
   if (NV) {
 #pragma unroll
@@ -76,26 +79,40 @@ __global__ void __launch_bounds__(512) shift_mix_kernel(const ShiftArgs a, int T
       if (NMIX) {
 #pragma unroll
         for (int m = 0; m < NMIX; ++m) get<VEC>(a.mu + (size_t)m * W + i, mus[m][q]);
-        if (a.second) get<VEC>(a.w2 + i, w2[q]);
       }
+      if (KEPT && a.second) get<VEC>(a.w2 + i, w2[q]);
     }
   }
   pdl_wait();
-  float x[N][VEC], o[N][VEC];                       // this token's row; the row before it, normed
+  float x[N][VEC], ahead[N][VEC], o[N][VEC];        // this token's row, the next one's; the row before it, normed
+  auto ask = [&](int at) {
+#pragma unroll
+    for (int q = 0; q < N; ++q) {
+      const int i = threadIdx.x * VEC + q * step;
+      if (i < W) get<VEC>(a.h + (size_t)at * W + i, ahead[q]);
+    }
+  };
+  if (NV && t < t_end) ask(t);
   bool carried = false;                             // o holds the normed row of token t - 1
   for (; t < t_end; ++t) {
-    if (a.token_seq && t >= row1) { find(t); carried = false; }
-    const bool before = a.token_seq && t > row0;
-    float* slot = a.token_seq && !before && id >= 0 ? a.prev + (size_t)id * W : nullptr;
+    if (shift && t >= row1) { find(t); carried = false; }
+    const bool before = shift && t > row0;
+    float* slot = shift && !before && id >= 0 ? a.prev + (size_t)id * W : nullptr;
     const float* hr = a.h + (size_t)t * W;
     // a second row is normed here: the one before (the CTA's first token), or the portion's last for its slot
     const float* other = before ? (carried ? nullptr : hr - W) : (slot && row1 - 1 > t ? a.h + (size_t)(row1 - 1) * W : nullptr);
     float y[N][VEC], held[N][VEC];
     float s0 = 0.f, s1 = 0.f;
+#pragma unroll
     for (int q = 0; NV ? q < N : threadIdx.x * VEC + q * step < W; ++q) {
       const int i = threadIdx.x * VEC + q * step, r = NV ? q : 0;
       if (i >= W) break;
-      get<VEC>(hr + i, x[r]);
+      if (NV) {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) x[r][e] = ahead[r][e];
+      } else {
+        get<VEC>(hr + i, x[r]);
+      }
       if (NV && slot) get<VEC>(slot + i, held[r]);
 #pragma unroll
       for (int e = 0; e < VEC; ++e) s0 = fmaf(x[r][e], x[r][e], s0);
@@ -105,13 +122,15 @@ __global__ void __launch_bounds__(512) shift_mix_kernel(const ShiftArgs a, int T
         for (int e = 0; e < VEC; ++e) s1 = fmaf(y[r][e], y[r][e], s1);
       }
     }
+    if (NV && t + 1 < t_end) ask(t + 1);
     // both sums over the block in one go, each in the same order
-    s0 = warp_sum(s0); s1 = warp_sum(s1);
+    s0 = warp_sum(s0);
+    if (other) s1 = warp_sum(s1);
     __syncthreads();
     if (lane == 0) { red[0][warp] = s0; red[1][warp] = s1; }
     __syncthreads();
     s0 = warp_sum(lane < nwarps ? red[0][lane] : 0.f) / (float)W;
-    s1 = warp_sum(lane < nwarps ? red[1][lane] : 0.f) / (float)W;
+    if (other) s1 = warp_sum(lane < nwarps ? red[1][lane] : 0.f) / (float)W;
     const float r = 1.f / sqrtf(s0 + a.eps), r2 = a.second ? 1.f / sqrtf(s0 + a.eps2) : 0.f, ro = 1.f / sqrtf(s1 + a.eps);
 #pragma unroll
     for (int q = 0; NV ? q < N : threadIdx.x * VEC + q * step < W; ++q) {
@@ -159,7 +178,7 @@ __global__ void __launch_bounds__(512) shift_mix_kernel(const ShiftArgs a, int T
       }
       if (a.plain) put<TO, VEC>((TO*)a.plain + (size_t)t * W + i, n);
       if (a.second) {
-        if (!NMIX) get<VEC>(a.w2 + i, w2[k]);
+        if (!KEPT) get<VEC>(a.w2 + i, w2[k]);
 #pragma unroll
         for (int e = 0; e < VEC; ++e) z[e] = x[k][e] * r2 * w2[k][e];
         put<TO, VEC>((TO*)a.second + (size_t)t * W + i, z);
@@ -314,18 +333,25 @@ lowrank_decay_few_kernel(const TI* __restrict__ z, long long ld, int rank, const
 template <typename TO>
 int launch_shift(const ShiftArgs& a, int T, bool vec, cudaStream_t s) {
   const int pieces = a.W / (vec ? 4 : 1);
-  const int threads = pieces >= 1024 && vec ? 512 : pieces >= 256 ? 256 : pieces >= 128 ? 128 : 64;
+  const int threads = pieces >= 512 && vec ? 512 : pieces >= 256 ? 256 : pieces >= 128 ? 128 : 64;
   const int nv = (pieces + threads - 1) / threads;
-  // long portions: two tokens a CTA, which share the norms of their rows and the shares of the mixes
-  const int per = T >= 1024 ? 2 : 1;
+  // long portions: as many tokens a CTA as fill the SMs once (two CTAs an SM where a thread has one piece of a row); they
+  // share the norms of their rows and what is read once a CTA
+  const int slots = 148 * (nv == 1 ? 2 : 1), per = vec && T >= 1024 ? (T + slots - 1) / slots : 1;
   const dim3 grid((T + per - 1) / per), block(threads);
-#define GO(V, NV, M) return launch_ex(shift_mix_kernel<TO, V, NV, M>, grid, block, 0, s, 1, a, T, per)
-  if (!vec) GO(1, 0, 0);
-  if (nv == 1 && a.nmix == 5) GO(4, 1, 5);
-  if (nv == 2 && a.nmix == 5) GO(4, 2, 5);
-  if (nv <= 2) GO(4, 2, 0);
-  if (nv <= 4) GO(4, 4, 0);
-  GO(4, 0, 0);
+#define GO(V, NV, M, S) return launch_ex(shift_mix_kernel<TO, V, NV, M, S>, grid, block, 0, s, 1, a, T, per)
+  if (!vec) GO(1, 0, 0, true);
+  if (!a.token_seq) {
+    if (nv == 1) GO(4, 1, 0, false);
+    if (nv == 2) GO(4, 2, 0, false);
+    if (nv <= 4) GO(4, 4, 0, false);
+    GO(4, 0, 0, false);
+  }
+  if (nv == 1 && a.nmix == 5) GO(4, 1, 5, true);
+  if (nv == 2 && a.nmix == 5) GO(4, 2, 5, true);
+  if (nv <= 2) GO(4, 2, 0, true);
+  if (nv <= 4) GO(4, 4, 0, true);
+  GO(4, 0, 0, true);
 #undef GO
 }
 

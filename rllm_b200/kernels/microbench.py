@@ -591,6 +591,8 @@ def cmd_timemix(a) -> None:
         h, prev = torch.randn(T, W, device=DEV), torch.zeros(batch, W, device=DEV)
         run([lambda: mix.shift_mix(h, w1, 1e-6, torch.bfloat16, mu, seq, cu, batch, slots, prev, second=(w2n, 1e-6))] * 4, 0,
             f"norm, shift and five mixes, second norm {what}", T * W * (4 + 6 * 2))
+        run([lambda: mix.shift_mix(h, w1, 1e-6, torch.bfloat16, plain=True, second=(w2n, 1e-6))] * 4, 0, f"two norms of one row {what}",
+            T * W * 8)
         run([lambda: ops.rmsnorm(h, w1, 1e-6, torch.bfloat16)] * 4, 0, f"  like: norm {what}", T * W * 6)
         z, wz, b0 = bf(T, rank), bf(C, rank), torch.randn(C, device=DEV)
         wt = wz.t().contiguous()
