@@ -295,8 +295,8 @@ RLLM_API int rllm_gla_decay(float* z, const float* bias, int T, int n, float tau
 }
 
 // proj [T, ld] (storage type): queries at q_off, keys at k_off (H x dim each), values at v_off (H x vdim).
-// alpha float [T, H * dim]: the decays. bonus float [H * dim] or null: the form with a bonus (top of this file). cu_q [S + 1]: row range of each sequence; state_slots [S] (-1: the state
-// starts at zero and is not kept). state float [slots, H, dim, vdim]. out float [T, H, vdim].
+// alpha float [T, H * dim]: the decays. bonus float [H * dim] or null: the form with a bonus (top of this file).
+// cu_q [S + 1]: row range of each sequence; state_slots [S] (-1: the state starts at zero and is not kept). state float [slots, H, dim, vdim]. out float [T, H, vdim].
 // chunk <= 0: every sequence's rows in one CTA per (head, 32 columns). chunk > 0: the three passes over chunks of
 // that many tokens; chunk_state: float [T / chunk + S, H, dim, vdim], chunk_decay: float [T / chunk + S, H, dim].
 RLLM_API int rllm_gla_scan(int dt, const void* proj, long long ld, int q_off, int k_off, int v_off, const float* alpha,

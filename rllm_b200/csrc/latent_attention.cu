@@ -630,8 +630,8 @@ latent_merge_kernel(const float* __restrict__ pacc, const float* __restrict__ pm
 // proj [T, ld]: head h's query at q_off + h * (dim + rot) as [dim plain | rot to rotate]; the down-projection
 // at dkv_off as [rank latent | rot shared key part]. table: float [T, dims/2, 2] (cos, sin). slots [T]: cache
 // row of each token (-1: do not write) or null. cache: rows of rank + rot. qfull: [T, H, rank + rot], of which
-// this writes the last rot of every head (null: no queries in proj). cq [T, cq_rank] (or null): proj's columns cq_off .. RMS-normed with
-// weight cq_w.
+// this writes the last rot of every head (null: no queries in proj). cq [T, cq_rank] (or null): proj's columns
+// cq_off .. RMS-normed with weight cq_w.
 RLLM_API int rllm_latent_prepare(int dt, const void* proj, long long ld, int q_off, int dkv_off, int T, int H, int dim,
                                  int rot, int rank, int dims, const float* wnorm, float eps, const float* table,
                                  const int* slots, void* cache, void* qfull, int cq_off, int cq_rank, const float* cq_w,

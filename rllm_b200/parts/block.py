@@ -6,7 +6,8 @@ every row, and before it the embedding's output again where it is given the embe
 layers begins with. `PostNormBlock` norms after the sum,
 h = norm(alpha h + sublayer(h)), the sublayers reading the stream itself; `OutputNormBlock` norms the sublayer's output
 alone, h += coef * norm(sublayer(h)), the sublayers again reading the stream itself. `ParallelBlock` has one norm whose
-output both sublayers read, or one norm each: h += mixer(n) + ffn(n), n = norm(h), or h += mixer(norm1(h)) + ffn(norm2(h)). `GatedPreNormBlock` is the pre-norm order with a
+output both sublayers read, or one norm each: h += mixer(n) + ffn(n), n = norm(h), or
+h += mixer(norm1(h)) + ffn(norm2(h)). `GatedPreNormBlock` is the pre-norm order with a
 gate on each sublayer's way into the stream: h += sigmoid(W_g n + b_g) * sublayer(n), n = norm(h), W_g a square matrix."""
 from __future__ import annotations
 
@@ -175,7 +176,8 @@ class OutputNormBlock(PostNormBlock):
 class ParallelBlock(Part):
     """h <- h + (mixer(n) + ffn(n)) with n = norm(h): one norm, both sublayers read its output, the feed-forward may
     be absent. With `ffn_norm` the feed-forward reads a norm of its own of the same h; the two are made in one pass where
-    they are not part of a product's kernel, and a mixer that norms the stream itself (`norms_stream`) makes both. Sublayers return their float outputs (a tensor, `Summands`, or `NormedSum` for a mixer whose members are
+    they are not part of a product's kernel, and a mixer that norms the stream itself (`norms_stream`) makes both.
+    Sublayers return their float outputs (a tensor, `Summands`, or `NormedSum` for a mixer whose members are
     normed before they are added); the sum of all of them and the residual sum are one float kernel. A mixer made
     of several mixers gets a tuple of cache layers. `names`: checkpoint sub-prefixes of mixer and feed-forward; the
     norm's weight is a tensor named by its `weight_name` under the block's prefix."""

@@ -126,7 +126,8 @@ class GluRoutedExperts(Part):
     `group_sum` (1 or 2) largest choice scores, only experts of the best `keep` groups can be chosen. `renorm`: weights
     divided by (their sum + `sum_eps`); `weight_scale` multiplies all weights. `shared`: a dense feed-forward every token
     uses (its tensors under `shared.`), added as it is, or times sigmoid(W_sg h) (`shared.sg`, one row) with `shared_gate`;
-    that row then stands under the router's in one product. Returns `Summands`: one float row per (token, chosen expert) and the shared expert's output; the block adds them."""
+    that row then stands under the router's in one product. Returns `Summands`: one float row per (token, chosen expert),
+    the shared expert's output and its gate logit; the block adds them."""
     graph_safe = True
     returns_output = True
 
